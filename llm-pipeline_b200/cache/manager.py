@@ -10,8 +10,8 @@ the scheduler decides.
 
 Layers with the same need form a *group* with pages of its own: one page id addresses the same
 page in every cache of the group (a tensor ``[num_pages, *spec.page_shape(page_size)]`` per cache:
-``[num_pages, 2, kv_heads, page_size, head_dim]`` for keys and values). A group whose layers see only a window of keys gives pages back as soon as every token
-in them has left the window (but for the pages of the first tokens where the spec keeps those visible); its block table then holds -1 there. Beside the pages, every live
+``[num_pages, 2, kv_heads, page_size, head_dim]`` for keys and values). A group whose layers see only a window or a chunk of keys gives pages back as soon as no later token
+sees a key in them (but for the pages of the first tokens where the spec keeps those visible); its block table then holds -1 there. Beside the pages, every live
 request owns a *slot*: an index into per-cache state tensors of fixed size per request, zeroed
 when the slot is handed out.
 """
@@ -188,10 +188,7 @@ class CacheManager:
     # -- pages -----------------------------------------------------------------------------
     def _first_needed_page(self, group: CacheGroup, start: int) -> int:
         """First logical page a step that starts at token ``start`` still has to hold."""
-        if group.spec.window is None:
-            return 0
-        lowest_key = max(0, start - group.spec.window + 1)
-        return lowest_key // self.page_size
+        return group.spec.first_key(start) // self.page_size
 
     def pages_short(self, req_id: Hashable, new_length: int) -> List[int]:
         """Per group, how many pages ``reserve(req_id, new_length)`` would have to take."""
@@ -245,7 +242,7 @@ class CacheManager:
             raise CacheError("a request's length cannot shrink")
         request.length = new_length
         for group in self.groups:
-            if group.spec.window is None:
+            if not group.spec.bounded:
                 continue
             table = group.tables[req_id]
             keep_from = self._first_needed_page(group, new_length)

@@ -4,7 +4,8 @@
 (``page_shape(page_size)``: the tensor of a cache is ``[num_pages, *page_shape]``), optionally its
 element type (default: the cache's), and ``window`` (None = every earlier token): pages whose
 tokens have all left the window may be given back while the request lives; with ``keep_first`` = n the
-first n tokens stay visible whatever the window, and their pages stay. Caches whose specs have
+first n tokens stay visible whatever the window, and their pages stay. ``chunk`` = n instead of a window: a token
+sees the keys of its own run of n tokens alone, the runs counted from position 0. Caches whose specs have
 the same ``group_key()`` share page ids and block tables. The manager, the memory budget and the
 benchmark read sizes from the spec alone (``elements_per_token``, ``bytes_per_token``).
 
@@ -31,6 +32,7 @@ class PagesSpec:
 
     window: Optional[int] = None
     keep_first: int = 0                          # tokens at a request's start that a window never leaves behind
+    chunk: Optional[int] = None                  # tokens see the keys of their own chunk of this many tokens
     dtype: Optional[torch.dtype] = None          # None: the element type the cache was made with
 
     def page_shape(self, page_size: int) -> Tuple[int, ...]:
@@ -38,7 +40,21 @@ class PagesSpec:
 
     def group_key(self):
         """Caches with equal keys form one group: one pool of page ids, one block table per request."""
-        return (type(self).__name__, self.page_shape(1), self.dtype, self.window, self.keep_first if self.window is not None else 0)
+        return (type(self).__name__, self.page_shape(1), self.dtype, self.window, self.keep_first if self.bounded else 0, self.chunk)
+
+    @property
+    def bounded(self) -> bool:
+        """Whether a request's pages may go back while it lives, because no later token sees their keys."""
+        return self.window is not None or self.chunk is not None
+
+    def first_key(self, position: int) -> int:
+        """The lowest key that the token at ``position`` sees (kept first tokens aside)."""
+        low = 0
+        if self.window is not None:
+            low = max(low, position - self.window + 1)
+        if self.chunk is not None:
+            low = max(low, position // self.chunk * self.chunk)
+        return low
 
     def elements_per_token(self) -> int:
         count = 1
@@ -69,6 +85,7 @@ class HeadRowPagesSpec(PagesSpec):
     row_size: int
     window: Optional[int] = None
     keep_first: int = 0
+    chunk: Optional[int] = None
 
     def page_shape(self, page_size: int) -> Tuple[int, ...]:
         return (self.num_kv_heads, page_size, self.row_size)

@@ -8,7 +8,8 @@ from .zupilorn import ZupilornConfig
 from .razelorn import RazelornConfig
 from .nufolix import NufolixConfig
 from .tupidra import TupidraConfig
+from .zasudra import ZasudraConfig
 
-__all__ = ["LayerSpec", "ModelConfig", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen3Config", "ZupilornConfig", "RazelornConfig", "NufolixConfig", "TupidraConfig",
+__all__ = ["LayerSpec", "ModelConfig", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen3Config", "ZupilornConfig", "RazelornConfig", "NufolixConfig", "TupidraConfig", "ZasudraConfig",
            "architecture_name", "load_config", "register_architecture", "resolve_config",
            "supported_architectures"]

@@ -4,14 +4,19 @@
 // With H query heads, G key/value heads (head h uses key/value head h / (H / G)), keys of d and values of dv entries,
 // for the token at position i and a key at position j <= i:
 //   seen(i, j) = i - j < window  or  j < keep_first                     (window 0: every j <= i)
+//   and, with a chunk size n > 0, i / n = j / n (whole division)
 //   s = (q . k) * scale;  s <- cap * tanh(s / cap) if cap > 0;  s <- s - slope[h] * (i - j)  if slopes are given
 //   p_j = exp(s_j) / (exp(sink[h]) + sum_seen exp(s_j))                 (without a sink: the plain softmax)
-//   o_h = sum_j p_j v_j;   o_h <- o_h * sigmoid(gate)  if a gate is given
+//   o_h = sum_j p_j v_j;   o_h <- o_h * sigmoid(gate)  if a gate is given (a number per channel, or one per head)
 // Scores, the cap, the bias, the softmax and the weighted sums are float32.
 //
 // capped_qkv_post: adds the projections' biases to the float32 product [q | k | v], divides every value head by its
 // root mean square (if asked), writes the queries in the compute type and the token's cache rows [k | v] per key/value
 // head into its page slot.
+//
+// capped_rows_post: the same step for designs that norm the whole rows of q and of k (before they are cut into heads) and
+// may rotate them: q and k divided by their root mean square times a weight per entry, the first rot entries of every head
+// rotated by the token's angles, values as projected (from their own columns, or the projected keys themselves).
 //
 // capped_attention (any sizes, float32 or bfloat16): a block per (token, key/value head, up to 8 heads of the group), a
 // warp per query head. Keys are walked in tiles of 32 aligned to key 0; tiles that hold no key the token sees are
@@ -62,6 +67,108 @@ __global__ void capped_qkv_post_kernel(const float* __restrict__ qkv, long qkv_t
     }
 }
 
+struct RowsPostArgs {
+    const float* proj; long proj_t;           // [tokens, q | k | ..]
+    const float* qw; const float* kw;         // [H d], [G d]: weights of the row norms
+    float eps;
+    const float* cos_t; const float* sin_t;   // [tokens, rot / 2] or null
+    int rot, interleaved;
+    void* q_out; long q_out_t;
+    const int* slots; void* pages;            // null: the queries alone
+    int page_size, H, G, d, dv;
+    int v_at;                                 // first column of the values
+};
+
+// Entry i of a row whose heads have d entries, normed by f and w, rotated within its head.
+__device__ __forceinline__ float rows_entry(const RowsPostArgs& a, const float* row, const float* w, float f, const float* cs, const float* sn,
+                                            int i) {
+    const float v = row[i] * f * w[i];
+    const int c = i % a.d;
+    if (c >= a.rot) return v;
+    const int half = a.rot >> 1;
+    const bool first = a.interleaved ? !(c & 1) : c < half;
+    const int at = a.interleaved ? c >> 1 : (first ? c : c - half);
+    const int other = i + (a.interleaved ? (first ? 1 : -1) : (first ? half : -half));
+    const float o = row[other] * f * w[other];
+    return first ? v * cs[at] - o * sn[at] : v * cs[at] + o * sn[at];
+}
+
+template <typename T> __device__ __forceinline__ void rows_store4(T* p, float4 v);
+template <> __device__ __forceinline__ void rows_store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void rows_store4<bf16>(bf16* p, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+}
+
+// A block per token. VEC: pieces of four entries (d, dv, rot multiples of 4, no rotation or the interleaved one).
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) capped_rows_post_kernel(const RowsPostArgs a) {
+    __shared__ float scratch[32];
+    pdl_wait();                                    // what the kernels before wrote is complete
+    pdl_trigger();
+    const int n = blockIdx.x;
+    const float* row = a.proj + (size_t)n * a.proj_t;
+    const int slot = a.pages ? a.slots[n] : -1;
+    const int nq = a.H * a.d, nk = a.pages ? a.G * a.d : 0, nv = a.pages ? a.G * a.dv : 0;
+    float sq = 0.f, sk = 0.f;
+    if (VEC) {
+        for (int i = threadIdx.x * 4; i < nq + nk; i += blockDim.x * 4) {
+            const float4 v = *reinterpret_cast<const float4*>(row + i);
+            const float s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+            if (i < nq) sq += s; else sk += s;
+        }
+    } else {
+        for (int i = threadIdx.x; i < nq + nk; i += blockDim.x) {
+            const float v = row[i];
+            if (i < nq) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
+        }
+    }
+    sq = block_sum(sq, scratch);
+    const float fq = 1.f / sqrtf(sq / (float)nq + a.eps);
+    float fk = 0.f;
+    if (nk > 0) {
+        sk = block_sum(sk, scratch);
+        fk = 1.f / sqrtf(sk / (float)nk + a.eps);
+    }
+    const int half = a.rot >> 1;
+    const float* cs = a.cos_t ? a.cos_t + (size_t)n * half : nullptr;
+    const float* sn = a.sin_t ? a.sin_t + (size_t)n * half : nullptr;
+    T* qo = reinterpret_cast<T*>(a.q_out) + (size_t)n * a.q_out_t;
+    const int rs = a.d + a.dv;
+    T* page_row = nullptr;
+    if (slot >= 0) page_row = reinterpret_cast<T*>(a.pages) + (((size_t)(slot / a.page_size) * a.G) * a.page_size + slot % a.page_size) * rs;
+    const size_t head_stride = (size_t)a.page_size * rs;
+    if (VEC) {
+        for (int i = threadIdx.x * 4; i < nq + nk + nv; i += blockDim.x * 4) {
+            if (i >= nq && !page_row) return;
+            if (i >= nq + nk) {                    // values as projected
+                const int j = i - nq - nk;
+                rows_store4(page_row + (size_t)(j / a.dv) * head_stride + a.d + j % a.dv, *reinterpret_cast<const float4*>(row + a.v_at + j));
+                continue;
+            }
+            const bool is_q = i < nq;
+            const int j = is_q ? i : i - nq, c = j % a.d;
+            const float f = is_q ? fq : fk;
+            float4 v = *reinterpret_cast<const float4*>(row + i);
+            const float4 w = *reinterpret_cast<const float4*>((is_q ? a.qw : a.kw) + j);
+            v = make_float4(v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w);
+            if (c < a.rot) {
+                const float2 co = *reinterpret_cast<const float2*>(cs + (c >> 1)), si = *reinterpret_cast<const float2*>(sn + (c >> 1));
+                v = make_float4(v.x * co.x - v.y * si.x, v.y * co.x + v.x * si.x, v.z * co.y - v.w * si.y, v.w * co.y + v.z * si.y);
+            }
+            if (is_q) rows_store4(qo + j, v);
+            else rows_store4(page_row + (size_t)(j / a.d) * head_stride + c, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < nq; i += blockDim.x) qo[i] = from_float<T>(rows_entry(a, row, a.qw, fq, cs, sn, i));
+        if (!page_row) return;
+        for (int i = threadIdx.x; i < nk; i += blockDim.x)
+            page_row[(size_t)(i / a.d) * head_stride + i % a.d] = from_float<T>(rows_entry(a, row + nq, a.kw, fk, cs, sn, i));
+        for (int i = threadIdx.x; i < nv; i += blockDim.x)
+            page_row[(size_t)(i / a.dv) * head_stride + a.d + i % a.dv] = from_float<T>(row[a.v_at + i]);
+    }
+}
+
 struct CappedArgs {
     const void* q; long q_t;                  // [tokens, H d]
     const void* pages;                        // [page, kv head, token in page, d + dv]
@@ -69,9 +176,10 @@ struct CappedArgs {
     const int* token_request; const int* positions;
     const float* slopes;                      // [H] or null
     const float* sink;                        // [H] or null
-    const float* gate; long gate_t;           // float32 [tokens, H dv] (a view) or null
+    const float* gate; long gate_t;           // float32 [tokens, H dv] (a view), [tokens, H] with gate_heads, or null
+    int gate_heads;
     void* out; long out_t;                    // [tokens, H dv]
-    int H, G, d, dv, page_size, window, keep;
+    int H, G, d, dv, page_size, window, keep, chunk;
     float scale, cap;
 };
 
@@ -95,7 +203,8 @@ __global__ void __launch_bounds__(CA_WARPS * 32) capped_attention_kernel(const C
     const int pos = a.positions[n];
     const int* table = a.tables + (size_t)a.token_request[n] * a.width;
     const T* pages = reinterpret_cast<const T*>(a.pages);
-    const int lo_w = a.window > 0 ? max(0, pos - a.window + 1) : 0;       // first key of the window
+    int lo_w = a.window > 0 ? max(0, pos - a.window + 1) : 0;             // first key of the window (and of the chunk)
+    if (a.chunk > 0) lo_w = max(lo_w, pos / a.chunk * a.chunk);
     const int keep_end = min(a.keep, lo_w);                               // kept keys before the window: [0, keep_end)
     float slope = 0.f, m_run = -INFINITY, l_run = 0.f;
     if (active) {
@@ -159,13 +268,13 @@ __global__ void __launch_bounds__(CA_WARPS * 32) capped_attention_kernel(const C
     if (!active) return;
     const float inv = 1.f / l_run;
     T* dst = reinterpret_cast<T*>(a.out) + (size_t)n * a.out_t + (size_t)h * dv;
-    const float* gate = a.gate ? a.gate + (size_t)n * a.gate_t + (size_t)h * dv : nullptr;
+    const float* gate = a.gate ? a.gate + (size_t)n * a.gate_t + (a.gate_heads ? (size_t)h : (size_t)h * dv) : nullptr;
 #pragma unroll
     for (int i = 0; i < NO; ++i) {
         const int c = lane + 32 * i;
         if (c < dv) {
             float v = o[i] * inv;
-            if (gate) v = v / (1.f + expf(-gate[c]));
+            if (gate) v = v / (1.f + expf(-gate[a.gate_heads ? 0 : c]));
             dst[c] = from_float<T>(v);
         }
     }
@@ -209,14 +318,33 @@ LLMP_API int llmp_capped_qkv_post(const float* qkv, long qkv_t, const void* bias
     return llmp_check_launch("capped_qkv_post");
 }
 
+LLMP_API int llmp_capped_rows_post(const float* proj, long proj_t, const float* qw, const float* kw, float eps, const float* cos_t,
+                                   const float* sin_t, int rot, int interleaved, void* q_out, int dtype, long q_out_t, const int* slots,
+                                   void* pages, int page_size, int v_at, int N, int H, int G, int d, int dv, cudaStream_t stream) {
+    if (N <= 0) return 0;
+    LLMP_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && dv > 0 && qw && (!pages || (kw && slots && page_size > 0)),
+                 "capped_rows_post: bad sizes heads=%d kv=%d dim=%d vdim=%d", H, G, d, dv);
+    LLMP_REQUIRE(rot >= 0 && rot <= d && rot % 2 == 0 && (rot == 0 || (cos_t && sin_t)), "capped_rows_post: a rotation of %d entries needs its tables", rot);
+    RowsPostArgs a;
+    a.proj = proj; a.proj_t = proj_t; a.qw = qw; a.kw = kw; a.eps = eps; a.cos_t = cos_t; a.sin_t = sin_t; a.rot = rot; a.interleaved = interleaved;
+    a.q_out = q_out; a.q_out_t = q_out_t; a.slots = slots; a.pages = pages; a.page_size = page_size; a.H = H; a.G = G; a.d = d; a.dv = dv; a.v_at = v_at;
+    const bool vec = d % 4 == 0 && dv % 4 == 0 && rot % 4 == 0 && (rot == 0 || interleaved) && proj_t % 4 == 0 && v_at % 4 == 0 && q_out_t % 4 == 0 &&
+                     ((size_t)proj | (size_t)qw | (size_t)kw | (size_t)cos_t | (size_t)sin_t | (size_t)q_out | (size_t)pages) % 16 == 0;
+    void (*kernel)(const RowsPostArgs) = dtype == LLMP_F32 ? (vec ? capped_rows_post_kernel<float, true> : capped_rows_post_kernel<float, false>)
+                                                           : (vec ? capped_rows_post_kernel<bf16, true> : capped_rows_post_kernel<bf16, false>);
+    llmp_launch_dependent(kernel, dim3(N), dim3(256), 0, stream, a);
+    return llmp_check_launch("capped_rows_post");
+}
+
 LLMP_API int llmp_capped_attention(const void* q, long q_t, const void* pages, int dtype, const int* tables, int width,
                                    const int* token_request, const int* positions, const float* slopes, const float* sink,
-                                   const float* gate, long gate_t, void* out, long out_t, int N, int H, int G, int d, int dv,
-                                   int page_size, int window, int keep, float scale, float cap, cudaStream_t stream) {
+                                   const float* gate, long gate_t, int gate_heads, void* out, long out_t, int N, int H, int G, int d,
+                                   int dv, int page_size, int window, int keep, int chunk, float scale, float cap, cudaStream_t stream) {
     if (N <= 0) return 0;
-    LLMP_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && dv > 0 && dv <= 512 && page_size > 0 && width > 0 && window >= 0 && keep >= 0,
+    LLMP_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && dv > 0 && dv <= 512 && page_size > 0 && width > 0 && window >= 0 && keep >= 0 && chunk >= 0,
                  "capped_attention: bad sizes heads=%d kv=%d dim=%d vdim=%d page=%d width=%d", H, G, d, dv, page_size, width);
     CappedArgs a;
+    a.gate_heads = gate_heads; a.chunk = chunk;
     a.q = q; a.q_t = q_t; a.pages = pages; a.tables = tables; a.width = width; a.token_request = token_request; a.positions = positions;
     a.slopes = slopes; a.sink = sink; a.gate = gate; a.gate_t = gate_t; a.out = out; a.out_t = out_t;
     a.H = H; a.G = G; a.d = d; a.dv = dv; a.page_size = page_size; a.window = window; a.keep = keep; a.scale = scale; a.cap = cap;

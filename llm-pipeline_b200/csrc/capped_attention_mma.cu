@@ -1,5 +1,6 @@
 // The capped window attention of capped_attention.cu over bfloat16 pages on the tensor cores (mma.sync m16n8k16, float32
-// accumulate), with the same arguments and result, for key sizes d and value sizes dv of 16, 32, 64 or 128.
+// accumulate), with the same arguments and result, for key sizes d and value sizes dv of 16, 32, 64 or 128, and for keys
+// and values of 48 or of 96.
 //
 // A block takes one tile of query rows of one request and one key/value head: CM_ROWS = 64 rows, a row being (token,
 // query head of the group) with the head running fastest, so the key/value tile it streams serves all query heads of
@@ -18,6 +19,11 @@
 // warp w takes keys 16 w to 16 w + 15 of it and keeps sums of its own; at the end the four meet in shared memory and warp 0
 // adds them in their order and stores. (With whole half tiles dealt out in turn, two warps worked while two waited at the
 // tile's barrier: 2.0 against 1.5 microseconds a tile at keys and values of 128.)
+//
+// Such steps can also cut a row's keys into segments of `segment_keys` (a multiple of the tile) with blocks of their own
+// (`segments` > 0, counted from the tile in which the row's keys begin, so they depend on the row's position alone):
+// every block leaves its sums (output, maximum, sum; float32) in scratch and counts itself, and the block of a tile that
+// counts last adds the segments in their order, applies the gate and stores. Nobody waits; the counters are left at zero.
 #include "common.cuh"
 
 #include <type_traits>
@@ -39,10 +45,12 @@ struct CappedMmaParams {
     const int* tile_tok0;
     const float* slopes;             // [heads] or null
     const float* sink;               // [heads] or null
-    const float* gate;               // float32 [tokens, heads dv] or null
+    const float* gate;               // float32 [tokens, heads dv] ([tokens, heads] with gate_heads) or null
+    float* scratch;                  // segments: [segment][token][head][dv + 2]
+    int* counters;                   // segments: one per (tile, kv head, chunk of heads), zero before and after a launch
     long q_stride, out_stride, gate_stride;
     int table_stride;
-    int nq, nkv, page_size, window, keep;
+    int nq, nkv, page_size, window, keep, chunk, gate_heads, segments, segment_keys, total_tokens;
     int heads_per_cta, tokens_per_cta, head_chunks, num_tiles, split, stages;
     float scale, cap;
 };
@@ -91,6 +99,13 @@ __device__ __forceinline__ unsigned cm_pack(float lo, float hi) {
 
 constexpr float CM_LOG2E = 1.4426950408889634f;
 
+// the lowest key (kept first tokens aside) that the token at `pos` sees
+__device__ __forceinline__ int cm_first_key(const CappedMmaParams& p, int pos) {
+    int lo = p.window > 0 ? pos - p.window + 1 : 0;
+    if (p.chunk > 0) lo = max(lo, pos / p.chunk * p.chunk);
+    return lo < 0 ? 0 : lo;
+}
+
 template <int D16, int V16>
 __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(const CappedMmaParams p) {
     extern __shared__ __align__(16) unsigned char cm_smem[];
@@ -129,20 +144,20 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
 
     // keys this block needs: the kept first tokens before its first token's window, then from that window's start to
     // the position of its last token
-    const int hi = pos0 + tok0 + ntok - 1;                       // last key (inclusive)
-    int lo = 0;
-    if (p.window > 0) {
-        lo = pos0 + tok0 - p.window + 1;
-        if (lo < 0) lo = 0;
-    }
+    int hi = pos0 + tok0 + ntok - 1;                             // last key (inclusive)
+    const int lo = cm_first_key(p, pos0 + tok0);
     const int keep_end = p.keep < lo ? p.keep : lo;              // kept keys that lie before the window: [0, keep_end)
     const int tile_lo = (lo / CM_KEYS) * CM_KEYS;
+    const int seg = blockIdx.y;
+    const int seg_needed = p.segments > 0 ? (hi - tile_lo) / p.segment_keys + 1 : 1;        // blocks that share this tile
+    if (seg >= seg_needed) return;
+    if (p.segments > 0) hi = min(hi, tile_lo + (seg + 1) * p.segment_keys - 1);
     // the walk: tiles 0, 64, .. below keep_end, then tile_lo, tile_lo + 64, .. up to hi
     auto next_tile = [&](int j0) {
         const int n = j0 + CM_KEYS;
         return (n >= keep_end && n < tile_lo) ? tile_lo : n;
     };
-    const int first_tile = keep_end > 0 ? 0 : tile_lo;
+    const int first_tile = seg > 0 ? tile_lo + seg * p.segment_keys : (keep_end > 0 ? 0 : tile_lo);     // segment 0 also has the kept tokens
 
     // query rows: row = token * hpc + head
     constexpr int QVEC = D / 8;
@@ -182,7 +197,7 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
     };
 
     // positions, slopes and sinks of this lane's two rows (row g and row g + 8 of the warp's 16); position -1: no such row
-    int row_pos[2];
+    int row_pos[2], row_lo[2];
     float slope2[2], m_run[2], l_run[2];
 #pragma unroll
     for (int h2 = 0; h2 < 2; ++h2) {
@@ -190,11 +205,12 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
         const int tl = row / hpc, h = row % hpc;
         const bool exists = tl < ntok && h < heads;
         row_pos[h2] = exists ? pos0 + tok0 + tl : -1;
+        row_lo[h2] = exists ? cm_first_key(p, pos0 + tok0 + tl) : 0;
         const int head = kvh * G + head0 + (exists ? h : 0);
         slope2[h2] = p.slopes ? p.slopes[head] * CM_LOG2E : 0.f;
         m_run[h2] = -INFINITY;
         l_run[h2] = 0.f;
-        if (p.sink && exists && (!split || warp == 0)) {
+        if (p.sink && exists && (!split || warp == 0) && seg == 0) {
             m_run[h2] = p.sink[head] * CM_LOG2E;
             l_run[h2] = t == 0 ? 1.f : 0.f;                     // the lanes of a quad add their sums at the end
         }
@@ -211,6 +227,8 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
     const bool warp_has_rows = warp_first_tok < ntok;            // a warp without rows only helps with the copies
     const int warp_hi_pos = pos0 + tok0 + (warp_last_tok < ntok ? warp_last_tok : ntok - 1);
     const int warp_lo_pos = pos0 + tok0 + (warp_first_tok < ntok ? warp_first_tok : ntok - 1);
+    const int warp_lo_first = cm_first_key(p, warp_lo_pos), warp_hi_first = cm_first_key(p, warp_hi_pos);
+    const bool plain = p.cap <= 0.f && !p.slopes;                // scores are scaled, nothing else
     const bf16* Qw = Qs + (size_t)(rw * 16 + (lane & 15)) * QSTRIDE + (lane >> 4) * 8;     // this lane's ldmatrix row of Q
     // the ring: stages - 1 tiles are under way beside the one at work (every round commits one group of copies, an empty
     // one once the walk's tiles are all asked for, so that the count of groups to wait for stays the same)
@@ -254,7 +272,9 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
             const int jh = j0 + kbase;
             if (jh > warp_hi_pos) return;                        // every row of this warp lies before these keys
             const bool kept = jh < p.keep;                       // kept first tokens stay in sight of every row
-            if (!kept && p.window > 0 && jh + NB * 8 - 1 < warp_lo_pos - p.window + 1) return;    // or sees none of them any more
+            if (!kept && jh + NB * 8 - 1 < warp_lo_first) return;       // or sees none of them any more
+            // every row of the warp sees every key of the part: no mask (rows that do not exist are never stored)
+            const bool all_seen = jh + NB * 8 - 1 <= warp_lo_pos && jh >= warp_hi_first;
             float s[NB][4];
 #pragma unroll
             for (int nb = 0; nb < NB; ++nb) s[nb][0] = s[nb][1] = s[nb][2] = s[nb][3] = 0.f;
@@ -277,15 +297,30 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
             for (int nb = 0; nb < NB; ++nb) {
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
-                    const int j = jh + nb * 8 + 2 * t + (c & 1);
-                    const int pos = row_pos[c >> 1];
-                    float v = p.cap > 0.f ? cap_log2 * cm_tanh(s[nb][c] * inv_cap) : s[nb][c] * scale_log2;
-                    v = fmaf(-slope2[c >> 1], (float)(pos - j), v);
-                    const bool ok = j <= pos && (p.window <= 0 || j >= pos - p.window + 1 || j < p.keep);
-                    v = ok ? v : -INFINITY;
-                    s[nb][c] = v;
-                    mx[c >> 1] = fmaxf(mx[c >> 1], v);
+                    if (plain) {
+                        s[nb][c] *= scale_log2;
+                    } else {
+                        const int j = jh + nb * 8 + 2 * t + (c & 1);
+                        const float v = p.cap > 0.f ? cap_log2 * cm_tanh(s[nb][c] * inv_cap) : s[nb][c] * scale_log2;
+                        s[nb][c] = fmaf(-slope2[c >> 1], (float)(row_pos[c >> 1] - j), v);
+                    }
                 }
+            }
+            if (!all_seen) {
+#pragma unroll
+                for (int nb = 0; nb < NB; ++nb) {
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) {
+                        const int j = jh + nb * 8 + 2 * t + (c & 1);
+                        const bool ok = j <= row_pos[c >> 1] && (j >= row_lo[c >> 1] || j < p.keep);
+                        s[nb][c] = ok ? s[nb][c] : -INFINITY;
+                    }
+                }
+            }
+#pragma unroll
+            for (int nb = 0; nb < NB; ++nb) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c) mx[c >> 1] = fmaxf(mx[c >> 1], s[nb][c]);
             }
             float alpha[2], m_use[2];
 #pragma unroll
@@ -363,8 +398,8 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
             *reinterpret_cast<float4*>(mine + 8 * V16) = make_float4(m_run[0], m_run[1], l_run[0], l_run[1]);
         }
         __syncthreads();
-        if (warp > 0) return;
-        for (int w = 0; w < 3; ++w) {
+        if (warp > 0 && p.segments <= 0) return;
+        for (int w = 0; w < 3 && warp == 0; ++w) {
             const float* theirs = xo + ((size_t)w * 32 + lane) * PER_LANE;
             const float4 ml = *reinterpret_cast<const float4*>(theirs + 8 * V16);
             const float om[2] = {ml.x, ml.y}, ol[2] = {ml.z, ml.w};
@@ -387,6 +422,60 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
             }
         }
     }
+    if (p.segments > 0) {
+        // this block's sums of its segment; the block that counts last adds them up (the whole block takes part)
+        __shared__ int last;
+        const size_t n = (size_t)(q_begin + tok0);
+        if (seg_needed > 1) {
+            if (warp == 0) {
+#pragma unroll
+                for (int h2 = 0; h2 < 2; ++h2) {
+                    if (row_pos[h2] < 0) continue;
+                    const int head = kvh * G + head0 + (g + 8 * h2) % hpc;
+                    float* dst = p.scratch + (((size_t)seg * p.total_tokens + n) * p.nq + head) * (DV + 2);
+#pragma unroll
+                    for (int nb = 0; nb < 2 * V16; ++nb) *reinterpret_cast<float2*>(dst + nb * 8 + 2 * t) = make_float2(o[nb][2 * h2], o[nb][2 * h2 + 1]);
+                    if (t == 0) *reinterpret_cast<float2*>(dst + DV) = make_float2(m_run[h2], l_run[h2]);
+                }
+                __threadfence();
+                __syncwarp();
+                if (lane == 0) {
+                    const int before = atomicAdd(&p.counters[blockIdx.x], 1);
+                    last = before == seg_needed - 1;
+                    if (last) p.counters[blockIdx.x] = 0;
+                    __threadfence();
+                }
+            }
+            __syncthreads();
+            if (!last) return;
+            constexpr int PAIRS = DV / 2;
+            for (int e = tid; e < heads * PAIRS; e += CM_THREADS) {
+                const int h = e / PAIRS, c = (e % PAIRS) * 2;
+                const int head = kvh * G + head0 + h;
+                const float* src = p.scratch + (n * p.nq + head) * (DV + 2);
+                const size_t step = (size_t)p.total_tokens * p.nq * (DV + 2);
+                float m = -INFINITY;
+                for (int s0 = 0; s0 < seg_needed; ++s0) m = fmaxf(m, __ldcg(src + s0 * step + DV));
+                float l = 0.f, a = 0.f, b = 0.f;
+                for (int s0 = 0; s0 < seg_needed; ++s0) {
+                    const float2 ml = __ldcg(reinterpret_cast<const float2*>(src + s0 * step + DV));
+                    const float2 v = __ldcg(reinterpret_cast<const float2*>(src + s0 * step + c));
+                    const float w = ml.x > -INFINITY ? cm_ex2(ml.x - m) : 0.f;
+                    l = fmaf(ml.y, w, l); a = fmaf(v.x, w, a); b = fmaf(v.y, w, b);
+                }
+                const float inv = l > 0.f ? 1.f / l : 0.f;
+                a *= inv; b *= inv;
+                if (p.gate) {
+                    const float* gate = p.gate + n * p.gate_stride + (p.gate_heads ? head : head * DV + c);
+                    a = a / (1.f + __expf(-gate[0]));
+                    b = b / (1.f + __expf(-gate[p.gate_heads ? 0 : 1]));
+                }
+                *reinterpret_cast<unsigned*>(p.out + n * p.out_stride + head * DV + c) = cm_pack(a, b);
+            }
+            return;
+        }
+        if (warp > 0) return;
+    }
 #pragma unroll
     for (int h2 = 0; h2 < 2; ++h2) {
         if (row_pos[h2] < 0) continue;
@@ -396,10 +485,11 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
         const size_t n = (size_t)(q_begin + tok0 + tl);
         const int col0 = (kvh * G + head0 + h) * DV + 2 * t;
         bf16* dst = p.out + n * p.out_stride + col0;
-        const float* gate = p.gate ? p.gate + n * p.gate_stride + col0 : nullptr;
+        const float* gate = p.gate && !p.gate_heads ? p.gate + n * p.gate_stride + col0 : nullptr;
+        const float head_gate = p.gate && p.gate_heads ? 1.f / (1.f + __expf(-p.gate[n * p.gate_stride + kvh * G + head0 + h])) : 1.f;
 #pragma unroll
         for (int nb = 0; nb < 2 * V16; ++nb) {
-            float a = o[nb][2 * h2] * inv, b = o[nb][2 * h2 + 1] * inv;
+            float a = o[nb][2 * h2] * inv * head_gate, b = o[nb][2 * h2 + 1] * inv * head_gate;
             if (gate) {
                 const float2 gv = *reinterpret_cast<const float2*>(gate + nb * 8);
                 a = a / (1.f + __expf(-gv.x));
@@ -410,7 +500,10 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
     }
 }
 
-bool cm_size_served(int n) { return n == 16 || n == 32 || n == 64 || n == 128; }
+bool cm_size_served(int d, int dv) {
+    auto any = [](int n) { return n == 16 || n == 32 || n == 64 || n == 128; };
+    return (any(d) && any(dv)) || (d == dv && (d == 48 || d == 96));
+}
 
 template <int D16, int V16>
 int launch_capped_mma(const CappedMmaParams& p, unsigned grid, cudaStream_t stream) {
@@ -419,19 +512,19 @@ int launch_capped_mma(const CappedMmaParams& p, unsigned grid, cudaStream_t stre
     // two buffers for prompts, so that two blocks share an SM; four for steps of single tokens, whose few blocks are each a
     // chain of copies that should be under way early
     CappedMmaParams q = p;
-    q.stages = (p.split && q_bytes + 4 * stage <= 200 * 1024) ? 4 : 2;
+    q.stages = (p.split && p.segments <= 0 && q_bytes + 4 * stage <= 200 * 1024) ? 4 : 2;
     size_t smem = q_bytes + q.stages * stage;
     const size_t meet = sizeof(float) * 3 * 32 * (size_t)(8 * V16 + 4);          // where the warps of a one-token tile meet
     if (smem < meet) smem = meet;
     // the kernel also has 2 KB of static shared memory: ask for the larger limit as soon as the two together pass 48 KB
     LLMP_ALLOW_SMEM((capped_attention_mma_kernel<D16, V16>), smem + 4096);
-    llmp_launch_dependent(capped_attention_mma_kernel<D16, V16>, dim3(grid), dim3(CM_THREADS), smem, stream, q);
+    llmp_launch_dependent(capped_attention_mma_kernel<D16, V16>, dim3(grid, p.segments > 0 ? p.segments : 1), dim3(CM_THREADS), smem, stream, q);
     return 0;
 }
 
 }  // namespace
 
-LLMP_API int llmp_capped_mma_supports(int d, int dv) { return cm_size_served(d) && cm_size_served(dv); }
+LLMP_API int llmp_capped_mma_supports(int d, int dv) { return cm_size_served(d, dv) ? 1 : 0; }
 
 // Query tokens per block for a group size: 64 rows of (token, head).
 LLMP_API int llmp_capped_mma_tokens_per_tile(int nq, int nkv) {
@@ -443,12 +536,17 @@ LLMP_API int llmp_capped_mma_tokens_per_tile(int nq, int nkv) {
 LLMP_API int llmp_capped_attention_mma(const void* q, long q_stride, void* out, long out_stride, const void* pages,
                                        const int* block_tables, int table_stride, const int* q_start, const int* ctx_len,
                                        const int* tile_req, const int* tile_tok0, int num_tiles, const float* slopes, const float* sink,
-                                       const float* gate, long gate_stride, int nq, int nkv, int d, int dv, int page_size, int window,
-                                       int keep, float scale, float cap, int split, cudaStream_t stream) {
+                                       const float* gate, long gate_stride, int gate_heads, int nq, int nkv, int d, int dv, int page_size,
+                                       int window, int keep, int chunk, float scale, float cap, int split, int segments, int segment_keys,
+                                       float* scratch, int* counters, int total_tokens, cudaStream_t stream) {
     if (num_tiles <= 0) return 0;
     LLMP_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0 && llmp_capped_mma_supports(d, dv) && page_size > 0 && window >= 0 && keep >= 0,
                  "capped_attention_mma: sizes heads=%d kv_heads=%d dim=%d vdim=%d are not served", nq, nkv, d, dv);
+    LLMP_REQUIRE(chunk >= 0 && segments >= 0 && segments <= 65535 && (segments == 0 || (split && scratch && counters && segment_keys > 0 &&
+                 segment_keys % CM_KEYS == 0 && (size_t)scratch % 8 == 0)), "capped_attention_mma: segments are for single tokens and need scratch and counters");
     CappedMmaParams p;
+    p.chunk = chunk; p.gate_heads = gate_heads; p.segments = segments; p.segment_keys = segment_keys; p.scratch = scratch; p.counters = counters;
+    p.total_tokens = total_tokens;
     p.q = (const bf16*)q; p.out = (bf16*)out; p.pages = (const bf16*)pages; p.block_tables = block_tables;
     p.q_start = q_start; p.ctx_len = ctx_len; p.tile_req = tile_req; p.tile_tok0 = tile_tok0;
     p.slopes = slopes; p.sink = sink; p.gate = gate; p.gate_stride = gate_stride;
@@ -463,7 +561,7 @@ LLMP_API int llmp_capped_attention_mma(const void* q, long q_stride, void* out, 
     p.stages = 2;
     LLMP_REQUIRE((long)num_tiles * nkv * p.head_chunks < (1L << 31), "capped_attention_mma: too many tiles");
     LLMP_REQUIRE((q_stride % 8) == 0 && (out_stride % 2) == 0 && ((size_t)q % 16) == 0 && ((size_t)pages % 16) == 0 &&
-                 ((size_t)out % 4) == 0 && (gate == nullptr || ((gate_stride % 2) == 0 && ((size_t)gate % 8) == 0)),
+                 ((size_t)out % 4) == 0 && (gate == nullptr || gate_heads || ((gate_stride % 2) == 0 && ((size_t)gate % 8) == 0)),
                  "capped_attention_mma: rows must be 16-byte aligned");
     const unsigned grid = (unsigned)(num_tiles * nkv * p.head_chunks);
     int rc = 1;
@@ -472,7 +570,11 @@ LLMP_API int llmp_capped_attention_mma(const void* q, long q_stride, void* out, 
     case DD:                                                             \
         switch (dv / 16) { CM_V(DD, 1) CM_V(DD, 2) CM_V(DD, 4) CM_V(DD, 8) } \
         break;
-    switch (d / 16) { CM_D(1) CM_D(2) CM_D(4) CM_D(8) }
+    switch (d / 16) {
+        CM_D(1) CM_D(2) CM_D(4) CM_D(8)
+        case 3: rc = launch_capped_mma<3, 3>(p, grid, stream); break;
+        case 6: rc = launch_capped_mma<6, 6>(p, grid, stream); break;
+    }
 #undef CM_D
 #undef CM_V
     if (rc) return rc;

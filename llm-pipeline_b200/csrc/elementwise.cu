@@ -34,6 +34,58 @@ LLMP_API int llmp_embedding(const int* ids, const void* table, int dtype, float*
 }
 
 // ------------------------------------------------------------------------------------------
+// Embedding with a second table whose row the previous and the current token choose:
+//   out[n, :] = table[ids[n], :] + bigram[row, :],  row = (prev * mul_prev + ids[n] * mul_cur) mod buckets,
+//   row = buckets (the last) for a request's first token.
+// The token before a step's first token of a request lies in the request's slot, two copies that take turns by the parity
+// of the last position written. The block of a request's first token in the step reads it and then notes the request's
+// last token of the step: the same copy when the step brings an even number of tokens.
+// ------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void embedding_bigram_kernel(const int* __restrict__ ids, const T* __restrict__ table, const T* __restrict__ bigram,
+                                        const int* __restrict__ q_start, const int* __restrict__ slots, const int* __restrict__ positions,
+                                        const int* __restrict__ token_request, int* __restrict__ state, long long mul_prev,
+                                        long long mul_cur, long long buckets, float* __restrict__ out, int H, int V) {
+    const int n = blockIdx.x;
+    const int id = ids[n], r = token_request[n], pos = positions[n];
+    const int begin = q_start[r];
+    long long row2 = buckets;
+    int* slot = state + (size_t)slots[r] * 2;
+    if (pos > 0) {
+        const int prev = n > begin ? ids[n - 1] : slot[(pos - 1) & 1];
+        row2 = ((long long)prev * mul_prev + (long long)id * mul_cur) % buckets;
+        if (row2 < 0) row2 += buckets;
+    }
+    if (n == begin) {
+        __syncthreads();                               // every thread has read the token before
+        if (threadIdx.x == 0) {
+            const int count = q_start[r + 1] - begin;
+            slot[(pos + count - 1) & 1] = ids[begin + count - 1];
+        }
+    }
+    const bool ok = id >= 0 && id < V;
+    const T* row = table + (size_t)(ok ? id : 0) * H;
+    const T* extra = bigram + (size_t)row2 * H;
+    float* dst = out + (size_t)n * H;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) dst[c] = ok ? to_float(row[c]) + to_float(extra[c]) : 0.f;
+}
+
+LLMP_API int llmp_embedding_bigram(const int* ids, const void* table, const void* bigram, int dtype, const int* q_start, const int* slots,
+                                   const int* positions, const int* token_request, int* state, long mul_prev, long mul_cur, long buckets,
+                                   float* out, int N, int H, int V, cudaStream_t stream) {
+    if (N <= 0) return 0;
+    LLMP_REQUIRE(H > 0 && V > 0 && buckets > 0, "embedding_bigram: bad sizes H=%d V=%d buckets=%ld", H, V, buckets);
+    const int threads = H >= 2048 && N <= 256 ? 512 : (H >= 1024 ? 256 : 128);
+    if (dtype == LLMP_F32)
+        embedding_bigram_kernel<float><<<N, threads, 0, stream>>>(ids, (const float*)table, (const float*)bigram, q_start, slots, positions,
+                                                                  token_request, state, mul_prev, mul_cur, buckets, out, H, V);
+    else
+        embedding_bigram_kernel<bf16><<<N, threads, 0, stream>>>(ids, (const bf16*)table, (const bf16*)bigram, q_start, slots, positions,
+                                                                 token_request, state, mul_prev, mul_cur, buckets, out, H, V);
+    return llmp_check_launch("embedding_bigram");
+}
+
+// ------------------------------------------------------------------------------------------
 // Rotary tables: cos/sin[n, j] = cos/sin(float(pos[n]) * inv_freq[j]) * scaling, float32.
 // ------------------------------------------------------------------------------------------
 __global__ void rope_tables_kernel(const int* __restrict__ pos, const float* __restrict__ inv_freq, float scaling,

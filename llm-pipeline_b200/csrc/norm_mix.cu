@@ -55,8 +55,9 @@ LLMP_API int llmp_embedding_norm(const int* ids, const void* table, int table_dt
 //   x = residual[r] + y
 //   if history:  history[index][r] = x;  x = sum_{j <= index} mix[j] * history[j][r]       (results of all layers so far)
 //   residual[r] = x                               (only without `rows`)
-//   out[m] = x * rsqrt(mean(x^2) + eps) * (offset + w)                     (if out)
+//   out[m] = x * rsqrt(mean(x^2) + eps) * (offset + w)                     (if out; without a weight: x itself)
 // One block per row; the row stays in shared memory between the passes. history is [slots][T][H] float32.
+// Steps that norm the addend and need neither history nor chosen rows take a form with the row in registers.
 // ------------------------------------------------------------------------------------------
 struct NormMixArgs {
     float* residual;
@@ -105,10 +106,81 @@ __global__ void add_norm_mix_kernel(const NormMixArgs a) {
         ss += x * x;
     }
     if (!a.out) return;
+    if (!a.w) {
+        for (int c = threadIdx.x; c < H; c += blockDim.x) store_dt(a.out, a.out_bf16, (size_t)m * H + c, xs[c]);
+        return;
+    }
     ss = block_sum(ss, scratch);
     const float rstd = rsqrtf(ss / (float)H + a.eps);
     for (int c = threadIdx.x; c < H; c += blockDim.x)
         store_dt(a.out, a.out_bf16, (size_t)m * H + c, xs[c] * rstd * (a.offset + load_dt(a.w, a.w_bf16, c)));
+}
+
+// The same for a normed addend without history and chosen rows, in 16-byte accesses with the row in registers: widths that
+// are multiples of 4 up to 4,096. The order of the sums follows from the width alone.
+constexpr int NX_THREADS = 256;
+constexpr int NX_PIECES = 4;
+
+__device__ __forceinline__ float4 nx_load4(const void* p, int is_bf16, size_t i4) {
+    if (!is_bf16) return reinterpret_cast<const float4*>(p)[i4];
+    const uint2 raw = reinterpret_cast<const uint2*>(p)[i4];
+    const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&raw.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
+    return make_float4(__low2float(lo), __high2float(lo), __low2float(hi), __high2float(hi));
+}
+
+__device__ __forceinline__ void nx_store4(void* p, int is_bf16, size_t i4, float4 v) {
+    if (!is_bf16) { reinterpret_cast<float4*>(p)[i4] = v; return; }
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    reinterpret_cast<uint2*>(p)[i4] = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+}
+
+__device__ __forceinline__ float nx_sum4(float4 v, float ss) { return fmaf(v.w, v.w, fmaf(v.z, v.z, fmaf(v.y, v.y, fmaf(v.x, v.x, ss)))); }
+
+__global__ void __launch_bounds__(NX_THREADS) add_normed_rows_kernel(const NormMixArgs a) {
+    __shared__ float scratch[32];
+    pdl_wait();                                    // what the kernels before wrote is complete
+    pdl_trigger();
+    const int H4 = a.H >> 2;
+    const size_t base = (size_t)blockIdx.x * H4;
+    float4 y[NX_PIECES], r[NX_PIECES];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NX_PIECES; ++j) {
+        const int i = threadIdx.x + j * NX_THREADS;
+        y[j] = r[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < H4) {
+            y[j] = nx_load4(a.delta, a.delta_bf16, base + i);
+            r[j] = reinterpret_cast<const float4*>(a.residual)[base + i];
+            ss = nx_sum4(y[j], ss);
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float f = rsqrtf(ss / (float)a.H + a.delta_eps);
+    ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NX_PIECES; ++j) {
+        const int i = threadIdx.x + j * NX_THREADS;
+        if (i < H4) {
+            const float4 w = nx_load4(a.delta_w, a.delta_w_bf16, i);
+            r[j].x += y[j].x * f * (a.delta_offset + w.x); r[j].y += y[j].y * f * (a.delta_offset + w.y);
+            r[j].z += y[j].z * f * (a.delta_offset + w.z); r[j].w += y[j].w * f * (a.delta_offset + w.w);
+            reinterpret_cast<float4*>(a.residual)[base + i] = r[j];
+            if (a.out && !a.w) nx_store4(a.out, a.out_bf16, base + i, r[j]);
+            ss = nx_sum4(r[j], ss);
+        }
+    }
+    if (!a.out || !a.w) return;
+    ss = block_sum(ss, scratch);
+    const float g = rsqrtf(ss / (float)a.H + a.eps);
+#pragma unroll
+    for (int j = 0; j < NX_PIECES; ++j) {
+        const int i = threadIdx.x + j * NX_THREADS;
+        if (i < H4) {
+            const float4 w = nx_load4(a.w, a.w_bf16, i);
+            nx_store4(a.out, a.out_bf16, base + i, make_float4(r[j].x * g * (a.offset + w.x), r[j].y * g * (a.offset + w.y),
+                                                              r[j].z * g * (a.offset + w.z), r[j].w * g * (a.offset + w.w)));
+        }
+    }
 }
 
 LLMP_API int llmp_add_norm_mix(float* residual, const void* delta, int delta_dtype, const void* delta_w, int delta_w_dtype,
@@ -118,7 +190,6 @@ LLMP_API int llmp_add_norm_mix(float* residual, const void* delta, int delta_dty
     if (M <= 0) return 0;
     LLMP_REQUIRE(H > 0 && (size_t)H * 4 <= 200 * 1024, "add_norm_mix: bad width %d", H);
     LLMP_REQUIRE(!history || (mix && index >= 0), "add_norm_mix: a history needs mixing weights and an index");
-    LLMP_REQUIRE(!out || w, "add_norm_mix: an output needs a norm weight");
     NormMixArgs a;
     a.residual = residual;
     a.delta = delta; a.delta_bf16 = delta_dtype == LLMP_BF16;
@@ -127,6 +198,12 @@ LLMP_API int llmp_add_norm_mix(float* residual, const void* delta, int delta_dty
     a.w = w; a.w_bf16 = w_dtype == LLMP_BF16; a.offset = offset; a.eps = eps;
     a.out = out; a.out_bf16 = out_dtype == LLMP_BF16;
     a.rows = rows; a.H = H;
+    auto aligned = [](const void* q, int bf) { return q == nullptr || ((size_t)q % (bf ? 8 : 16)) == 0; };
+    if (delta && delta_w && !history && !rows && H % 4 == 0 && H <= 4 * NX_THREADS * NX_PIECES && aligned(residual, 0) &&
+        aligned(delta, a.delta_bf16) && aligned(delta_w, a.delta_w_bf16) && aligned(w, a.w_bf16) && aligned(out, a.out_bf16)) {
+        llmp_launch_dependent(add_normed_rows_kernel, dim3(M), dim3(NX_THREADS), 0, stream, a);
+        return llmp_check_launch("add_norm_mix");
+    }
     const size_t smem = (size_t)H * sizeof(float);
     LLMP_ALLOW_SMEM(add_norm_mix_kernel, smem);
     // few rows (a decode step): as many threads as the row has pairs of entries, so that a thread's loads are few

@@ -2,14 +2,16 @@
 //   route_topk:      router logits in float32 (float32 copy of the router matrix, the token's row as stored); scores by
 //                    sigmoid (each logit alone) or softmax (over all router outputs); the `top` largest of
 //                    score (+ a correction per router output, if given); a chosen expert's weight is its score
-//                    without the correction. A further row of the matrix, if asked for, gives a gate per token:
+//                    without the correction. Or the `top` largest logits, and a softmax over those alone. A bias per
+//                    router output joins the logits, if given. A further row of the matrix, if asked for, gives a gate per token:
 //                    sigmoid of its logit.
 //   expert_gate_up:  per (token, choice), with w the choice's weight, by the form of the expert:
 //                    clamped:  g = min(w (Wg h), limit), u = clamp(w (Wu h), -limit, limit), y = g sigmoid(1.702 g) (u + 1)
 //                              (the weight scales the expert's input; the first products are linear, so it is applied to
 //                              their float32 sums);
 //                    silu:     y = w silu(Wg h) (Wu h) (the weight scales the expert's output; the last product is
-//                              linear, so it is applied to the float32 activation before it is rounded).
+//                              linear, so it is applied to the float32 activation before it is rounded);
+//                    relu_squared:  y = w max(Wu h, 0)^2 (no gate matrix; the weight scales the expert's output).
 //   expert_down:     out[token] = sum over the token's choices, in their order, of Wd y (float32). A choice whose id is
 //                    not below the number of experts with matrices is an identity expert: it adds w h.
 // These kernels read an expert's rows once per token that chose it (a warp per output row): the form for the few
@@ -18,8 +20,11 @@
 #include "common.cuh"
 
 __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const float* __restrict__ wr, int top, int* __restrict__ ids,
-                                  float* __restrict__ wts, int Hd, int E, int softmax, const float* __restrict__ correction,
-                                  float* __restrict__ gate) {
+                                  float* __restrict__ wts, int Hd, int E, int mode, const float* __restrict__ bias,
+                                  const float* __restrict__ correction, float* __restrict__ gate) {
+    pdl_wait();                                    // what the kernels before wrote is complete
+    pdl_trigger();
+    const bool softmax = mode == 1;
     extern __shared__ float route_smem[];
     float* logits = route_smem;                              // [E + 1]: logits, then what the choice goes by
     float* score = route_smem + E + 1;                       // [E]: softmax scores (softmax only)
@@ -42,7 +47,7 @@ __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const 
         }
         for (; i < Hd; i += 32) acc[0] = fmaf(row[i], w[i], acc[0]);
         const float s = warp_sum(((acc[0] + acc[1]) + (acc[2] + acc[3])) + ((acc[4] + acc[5]) + (acc[6] + acc[7])));
-        if (lane == 0) logits[e] = s;
+        if (lane == 0) logits[e] = (bias && e < E) ? s + bias[e] : s;
     }
     __syncthreads();
     if (warp == 0) {
@@ -73,6 +78,7 @@ __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const 
             __syncwarp();
         }
         const bool by_score = softmax || correction;
+        float first = 0.f, total = 0.f;                      // mode 2: the largest logit, and the sum of the chosen exponentials
         for (int k = 0; k < top; ++k) {
             float best = -INFINITY;
             int at = -1;
@@ -85,31 +91,47 @@ __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const 
             }
             if (lane == 0) {
                 ids[(size_t)n * top + k] = at;
-                wts[(size_t)n * top + k] = by_score ? score[at] : 1.f / (1.f + expf(-best));
+                float w;
+                if (mode == 2) {
+                    if (k == 0) first = best;
+                    w = expf(best - first);
+                    total += w;
+                } else {
+                    w = by_score ? score[at] : 1.f / (1.f + expf(-best));
+                }
+                wts[(size_t)n * top + k] = w;
                 logits[at] = -INFINITY;
             }
             __syncwarp();
         }
+        if (mode == 2) {
+            total = __shfl_sync(0xffffffffu, total, 0);
+            for (int k = lane; k < top; k += 32) wts[(size_t)n * top + k] /= total;
+        }
     }
 }
 
-// softmax: 0 sigmoid scores, 1 softmax over the E router outputs. correction: float32 [E] or null. gate: float32 [N] or
+// mode: 0 sigmoid scores, 1 softmax over the E router outputs, 2 softmax over the chosen logits. bias: float32 [E] or null. correction: float32 [E] or null. gate: float32 [N] or
 // null; when given, w_router has E + 1 rows and gate[n] = sigmoid(row E . h[n]).
 LLMP_API int llmp_route_topk(const void* h, int h_dtype, const float* w_router, int top, int* ids, float* wts, int N, int Hd, int E,
-                             int softmax, const float* correction, float* gate, cudaStream_t stream) {
+                             int mode, const float* bias, const float* correction, float* gate, cudaStream_t stream) {
     if (N <= 0) return 0;
+    LLMP_REQUIRE(mode >= 0 && mode <= 2 && (mode != 2 || !correction), "route_topk: mode %d", mode);
     LLMP_REQUIRE(E > 0 && top > 0 && top <= E && Hd > 0 && E <= 8192, "route_topk: bad sizes experts=%d top=%d width=%d", E, top, Hd);
     const size_t smem = (size_t)(2 * E + 1 + Hd) * sizeof(float);
     LLMP_REQUIRE(smem <= 200 * 1024, "route_topk: a row of %d entries does not fit shared memory", Hd);
     LLMP_ALLOW_SMEM(route_topk_kernel, smem);
     // few rows (a decode step): a warp per expert, so that the router matrix is read by many warps at once
-    route_topk_kernel<<<N, N <= 64 ? 1024 : 256, smem, stream>>>(h, h_dtype == LLMP_BF16, w_router, top, ids, wts, Hd, E, softmax,
-                                                                  correction, gate);
+    llmp_launch_dependent(route_topk_kernel, dim3(N), dim3(N <= 64 ? 1024 : 256), smem, stream, h, (int)(h_dtype == LLMP_BF16), w_router,
+                          top, ids, wts, Hd, E, mode, bias, correction, gate);
     return llmp_check_launch("route_topk");
 }
 
-// form 0: clamped, the weight on the input; form 1: silu(g) u, the weight on the output
+// form 0: clamped, the weight on the input; form 1: silu(g) u, the weight on the output; form 2: max(u, 0)^2 without a
+// gate, the weight on the output
+#define EXPERT_FORM_UNGATED 2
 __device__ __forceinline__ float expert_act(float g, float u, float w, float limit, int form) {
+    if (form == EXPERT_FORM_UNGATED) { u = fmaxf(u, 0.f); return w * (u * u); }
     if (form == 1) return w * (g / (1.f + expf(-g))) * u;
     g = fminf(w * g, limit);
     u = fminf(fmaxf(w * u, -limit), limit);
@@ -132,12 +154,15 @@ __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
-// grid (pairs, ceil(F / 8)): a warp per row of the expert's gate and up matrices (w_gu[e] = [gate rows; up rows]).
+// grid (pairs, ceil(F / 8)): a warp per row of the expert's gate and up matrices (w_gu[e] = [gate rows; up rows], or the up
+// rows alone for the form without a gate).
 // VEC: the rows' length is a multiple of 8; a lane then takes 8 consecutive entries a step, in 16-byte loads.
-template <typename T, bool VEC>
+template <typename T, bool VEC, bool GATED>
 __global__ void expert_gate_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gu, const int* __restrict__ ids,
                                       const float* __restrict__ wts, float limit, T* __restrict__ y, int top, int Hd, int F,
                                       int form, int E) {
+    pdl_wait();
+    pdl_trigger();
     const int pair = blockIdx.x;
     const int f = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
@@ -145,30 +170,30 @@ __global__ void expert_gate_up_kernel(const T* __restrict__ h, const T* __restri
     const int e = ids[pair];
     if (e >= E) return;                                      // an identity expert has no matrices
     const T* x = h + (size_t)(pair / top) * Hd;
-    const T* wg = w_gu + ((size_t)e * 2 * F + f) * Hd;
-    const T* wu = wg + (size_t)F * Hd;
+    const T* wg = w_gu + ((size_t)e * (GATED ? 2 : 1) * F + f) * Hd;
+    const T* wu = GATED ? wg + (size_t)F * Hd : wg;
     float g = 0.f, u = 0.f;
     if (VEC) {
 #pragma unroll 2
         for (int i = lane * 8; i < Hd; i += 256) {
             float xv[8], a[8], b[8];
             load8(x + i, xv);
-            load8(wg + i, a);
+            if (GATED) load8(wg + i, a);
             load8(wu + i, b);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                g = fmaf(xv[j], a[j], g);
+                if (GATED) g = fmaf(xv[j], a[j], g);
                 u = fmaf(xv[j], b[j], u);
             }
         }
     } else {
         for (int i = lane; i < Hd; i += 32) {
             const float xv = to_float(x[i]);
-            g = fmaf(xv, to_float(wg[i]), g);
+            if (GATED) g = fmaf(xv, to_float(wg[i]), g);
             u = fmaf(xv, to_float(wu[i]), u);
         }
     }
-    g = warp_sum(g);
+    if (GATED) g = warp_sum(g);
     u = warp_sum(u);
     if (lane == 0) y[(size_t)pair * F + f] = from_float<T>(expert_act(g, u, wts[pair], limit, form));
 }
@@ -178,6 +203,8 @@ template <typename T, bool VEC>
 __global__ void expert_down_kernel(const T* __restrict__ y, const T* __restrict__ w_down, const int* __restrict__ ids,
                                    float* __restrict__ out, int top, int Hd, int F, const T* __restrict__ h,
                                    const float* __restrict__ wts, int E) {
+    pdl_wait();
+    pdl_trigger();
     const int n = blockIdx.x;
     const int c = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
@@ -217,13 +244,15 @@ LLMP_API int llmp_expert_rows(const void* h, const void* w_gu, const void* w_dow
     LLMP_REQUIRE((F + 7) / 8 <= 65535 && (Hd + 7) / 8 <= 65535, "expert_rows: too wide");
     dim3 g1(N * top, (F + 7) / 8), g2(N, (Hd + 7) / 8);
     const bool aligned = ((size_t)h | (size_t)w_gu | (size_t)w_down | (size_t)y) % 16 == 0;
-    const bool v1 = aligned && Hd % 8 == 0, v2 = aligned && F % 8 == 0;
+    const bool v1 = aligned && Hd % 8 == 0, v2 = aligned && F % 8 == 0, gated = form != EXPERT_FORM_UNGATED;
 #define LLMP_EXPERT_ROWS(T)                                                                                                        \
     do {                                                                                                                           \
-        if (v1) expert_gate_up_kernel<T, true><<<g1, 256, 0, stream>>>((const T*)h, (const T*)w_gu, ids, wts, limit, (T*)y, top, Hd, F, form, E);  \
-        else expert_gate_up_kernel<T, false><<<g1, 256, 0, stream>>>((const T*)h, (const T*)w_gu, ids, wts, limit, (T*)y, top, Hd, F, form, E);    \
-        if (v2) expert_down_kernel<T, true><<<g2, 256, 0, stream>>>((const T*)y, (const T*)w_down, ids, out, top, Hd, F, (const T*)h, wts, E);                 \
-        else expert_down_kernel<T, false><<<g2, 256, 0, stream>>>((const T*)y, (const T*)w_down, ids, out, top, Hd, F, (const T*)h, wts, E);                   \
+        void (*up)(const T*, const T*, const int*, const float*, float, T*, int, int, int, int, int);                              \
+        if (gated) up = v1 ? expert_gate_up_kernel<T, true, true> : expert_gate_up_kernel<T, false, true>;                         \
+        else up = v1 ? expert_gate_up_kernel<T, true, false> : expert_gate_up_kernel<T, false, false>;                             \
+        llmp_launch_dependent(up, g1, dim3(256), 0, stream, (const T*)h, (const T*)w_gu, ids, wts, limit, (T*)y, top, Hd, F, form, E);  \
+        llmp_launch_dependent(v2 ? expert_down_kernel<T, true> : expert_down_kernel<T, false>, g2, dim3(256), 0, stream,           \
+                              (const T*)y, (const T*)w_down, ids, out, top, Hd, F, (const T*)h, wts, E);                           \
     } while (0)
     if (dtype == LLMP_F32) LLMP_EXPERT_ROWS(float);
     else LLMP_EXPERT_ROWS(bf16);
@@ -238,7 +267,7 @@ LLMP_API int llmp_expert_rows(const void* h, const void* w_gu, const void* w_dow
 //       expert's last pair and the next multiple of 64 hold -1. Which place within its expert's run a pair gets
 //       depends on the order of atomic adds, but a row's result does not depend on its place.
 //   grouped products: a block takes a tile of 64 sorted rows and 64 output columns, its four warps 16 rows each.
-//       First product: rows gathered from h by pair, against the expert's gate rows and up rows of the same columns,
+//       First product: rows gathered from h by pair, against the expert's gate rows (if it has them) and up rows of the same columns,
 //       with the activation in the epilogue (y, bfloat16, in sorted order). Second product: y against the expert's
 //       down rows, written as float32 at the pair's own place.
 //   combine: out[token] = sum of its pairs' rows in the order of its choices.
@@ -306,8 +335,8 @@ struct GroupedArgs {
     float limit;
 };
 
-// GATED: the first product (two weight tiles, activation); else the second.
-template <bool GATED>
+// FIRST: the first product (with the activation; GATED: two weight tiles); else the second.
+template <bool FIRST, bool GATED>
 __global__ void __launch_bounds__(128) moe_grouped_kernel(const GroupedArgs a) {
     // two stages of [A tile | weight tile(s)], each tile [64][GX_STRIDE]: the copies of the next K step run under the
     // products of this one
@@ -339,7 +368,7 @@ __global__ void __launch_bounds__(128) moe_grouped_kernel(const GroupedArgs a) {
             const int row = v / (GX_K / 8), c = (v % (GX_K / 8)) * 8;
             const int pair = row_pair[row];
             const bool ok = pair >= 0 && k0 + c < a.K;
-            const size_t src_row = GATED ? (size_t)(pair / a.top) : (size_t)(row0 + row);
+            const size_t src_row = FIRST ? (size_t)(pair / a.top) : (size_t)(row0 + row);
             gx_cp_async_16(As + row * GX_STRIDE + c, ok ? a.a + src_row * a.K + k0 + c : a.a, ok);
             const bool okw = col0 + row < a.cols_total && k0 + c < a.K;
             gx_cp_async_16(Bs + row * GX_STRIDE + c, okw ? wg + (size_t)row * a.K + k0 + c : a.w, okw);
@@ -384,14 +413,15 @@ __global__ void __launch_bounds__(128) moe_grouped_kernel(const GroupedArgs a) {
         const int row = warp * 16 + g + 8 * h2;
         const int pair = row_pair[row];
         if (pair < 0) continue;
-        const float w = GATED ? a.wts[pair] : 0.f;
+        const float w = FIRST ? a.wts[pair] : 0.f;
 #pragma unroll
         for (int nb = 0; nb < 8; ++nb) {
 #pragma unroll
             for (int c2 = 0; c2 < 2; ++c2) {
                 const int col = col0 + nb * 8 + 2 * t + c2;
                 if (col >= a.cols_total) continue;
-                if (GATED) a.y[(size_t)(row0 + row) * a.cols_total + col] = __float2bfloat16_rn(expert_act(cg[nb][2 * h2 + c2], cu[GATED ? nb : 0][2 * h2 + c2], w, a.limit, a.form));
+                // without a gate the up rows are the only weight tile: their sums are cg
+                if (FIRST) a.y[(size_t)(row0 + row) * a.cols_total + col] = __float2bfloat16_rn(expert_act(cg[nb][2 * h2 + c2], GATED ? cu[GATED ? nb : 0][2 * h2 + c2] : cg[nb][2 * h2 + c2], w, a.limit, a.form));
                 else a.out[(size_t)pair * a.cols_total + col] = cg[nb][2 * h2 + c2];
             }
         }
@@ -445,11 +475,17 @@ LLMP_API int llmp_expert_grouped(const void* h, const void* w_gu, const void* w_
     LLMP_REQUIRE(!combine || pair_out, "expert_grouped: the sum over a token's choices needs its scratch");
     a.a = (const bf16*)h; a.w = (const bf16*)w_gu; a.K = Hd; a.cols_total = F; a.out = nullptr;
     const size_t smem_gated = sizeof(bf16) * 2 * 3 * GX_ROWS * GX_STRIDE, smem_plain = sizeof(bf16) * 2 * 2 * GX_ROWS * GX_STRIDE;
-    LLMP_ALLOW_SMEM(moe_grouped_kernel<true>, smem_gated);
-    moe_grouped_kernel<true><<<dim3(tiles_max, (F + GX_COLS - 1) / GX_COLS), 128, smem_gated, stream>>>(a);
+    const dim3 first_grid(tiles_max, (F + GX_COLS - 1) / GX_COLS);
+    if (form != EXPERT_FORM_UNGATED) {
+        LLMP_ALLOW_SMEM((moe_grouped_kernel<true, true>), smem_gated);
+        moe_grouped_kernel<true, true><<<first_grid, 128, smem_gated, stream>>>(a);
+    } else {
+        LLMP_ALLOW_SMEM((moe_grouped_kernel<true, false>), smem_plain);
+        moe_grouped_kernel<true, false><<<first_grid, 128, smem_plain, stream>>>(a);
+    }
     a.a = (const bf16*)y; a.w = (const bf16*)w_down; a.K = F; a.cols_total = Hd; a.out = combine ? pair_out : out;
-    LLMP_ALLOW_SMEM(moe_grouped_kernel<false>, smem_plain);
-    moe_grouped_kernel<false><<<dim3(tiles_max, (Hd + GX_COLS - 1) / GX_COLS), 128, smem_plain, stream>>>(a);
+    LLMP_ALLOW_SMEM((moe_grouped_kernel<false, false>), smem_plain);
+    moe_grouped_kernel<false, false><<<dim3(tiles_max, (Hd + GX_COLS - 1) / GX_COLS), 128, smem_plain, stream>>>(a);
     if (combine) {
         const size_t total = (size_t)N * Hd;
         moe_combine_kernel<<<(unsigned)((total + 255) / 256), 256, 0, stream>>>(pair_out, out, top, Hd, total, ids, wts, (const bf16*)h, E);

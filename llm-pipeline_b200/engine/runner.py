@@ -449,7 +449,7 @@ class ModelRunner:
             torch.cuda.synchronize(self.device)
             piece.graph = torch.cuda.CUDAGraph()
             with torch.cuda.graph(piece.graph, pool=pool):
-                stream = model.begin(ctx) if k == 0 else ResidualStream(piece.inlet, slot.history)
+                stream = model.begin(ctx, self._views) if k == 0 else ResidualStream(piece.inlet, slot.history)
                 if k == 0:
                     slot.history = stream.history        # layer results that a model with a depth mix keeps: one buffer for all pieces
                 model.run_layers(ctx, self._views, stream, first, end)
@@ -505,7 +505,7 @@ class ModelRunner:
             buf[at:at + R] = mapping
             at += R
             lens = slot.table_lens[g]
-            windowed = group.spec.window is not None
+            windowed = group.spec.bounded
             for r, table in enumerate(tables):
                 if windowed or len(table) != lens[r]:
                     n = min(width, len(table))

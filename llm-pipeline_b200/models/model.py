@@ -48,6 +48,8 @@ class Model:
         self._owner: Dict[int, int] = {}
         for i, entry in enumerate(self.schedule):
             self._owner.setdefault(entry.cache, i)
+        # an embedding that carries something from token to token has a cache id of its own, after those of the layers
+        self.embedding_cache = len(self._owner) if self.embedding.state_spec() is not None else None
         # one mixer of every group whose members answer ``graph_key`` alike (36 equal attention layers: one question)
         self._key_mixers = list({block.mixer.graph_key_group(): block.mixer
                                  for block in (self.blocks[e.layer] for e in self.schedule)}.values())
@@ -84,12 +86,15 @@ class Model:
         return min(limits) if limits else None
 
     def cache_specs(self) -> List[Tuple[Optional[PagesSpec], Optional[StateSpec]]]:
-        """Per cache id, what the layer that owns it asks of the cache manager."""
+        """Per cache id, what the layer that owns it asks of the cache manager; last, what the embedding asks, if it
+        carries something from token to token."""
         count = max((e.cache for e in self.schedule), default=-1) + 1
         specs: List[Tuple[Optional[PagesSpec], Optional[StateSpec]]] = [(None, None)] * count
         for cache_id, index in self._owner.items():
             block = self.blocks[self.schedule[index].layer]
             specs[cache_id] = (block.mixer.cache_spec(), block.state_spec())
+        if self.embedding_cache is not None:
+            specs.append((None, self.embedding.state_spec()))
         return specs
 
     # -- weights ---------------------------------------------------------------------------
@@ -130,16 +135,19 @@ class Model:
     def forward(self, ctx, caches) -> ResidualStream:
         """Run every scheduled layer on the step's tokens. ``caches.view(cache_id, writes)`` gives
         the ``LayerCache`` of an execution."""
-        stream = self.begin(ctx)
+        stream = self.begin(ctx, caches)
         self.run_layers(ctx, caches, stream, 0, len(self.schedule))
         return stream
 
-    def begin(self, ctx) -> ResidualStream:
+    def begin(self, ctx, caches) -> ResidualStream:
         """What comes before the first layer: the position tables of the step and the embedded tokens."""
         begin_step()
         with nvtx_range("positions and embedding"):
             ctx.position_tables = {name: part.tables(ctx) for name, part in self.positions.items()}
-            residual = self.embedding.forward(ctx)
+            if self.embedding_cache is None:
+                residual = self.embedding.forward(ctx)
+            else:
+                residual = self.embedding.forward_with_state(ctx, caches.view(self.embedding_cache, writes=True).state)
             history = None
             if self.history_slots:
                 history = torch.empty((self.history_slots,) + tuple(residual.shape), dtype=torch.float32, device=residual.device)

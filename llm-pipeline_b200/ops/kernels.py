@@ -37,6 +37,7 @@ def dtype_code(dtype: torch.dtype) -> int:
 
 _SIGNATURES = {
     "llmp_embedding": [_P, _P, _I, _P, _I, _I, _I, _F, _P],
+    "llmp_embedding_bigram": [_P, _P, _P, _I, _P, _P, _P, _P, _P, _L, _L, _L, _P, _I, _I, _I, _P],
     "llmp_rope_tables": [_P, _P, _F, _P, _P, _I, _I, _P],
     "llmp_add_rmsnorm": [_P, _P, _P, _I, _P, _I, _F, _P, _I, _P, _I, _I, _P],
     "llmp_qkv_post": [_P, _I, _P, _I, _P, _P, _I, _F, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
@@ -69,14 +70,16 @@ _SIGNATURES = {
                                   _I, _P, _P, _P],
     "llmp_latent_rows_post": [_P, _L, _P, _L, _I, _I, _I, _I, _P, _I, _F, _P, _P, _I, _I, _P, _I, _L, _P, _P, _I, _P],
     "llmp_capped_qkv_post": [_P, _L, _P, _I, _F, _I, _P, _I, _L, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-    "llmp_capped_attention": [_P, _L, _P, _I, _P, _I, _P, _P, _P, _P, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
-    "llmp_capped_attention_mma": [_P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P],
+    "llmp_capped_rows_post": [_P, _L, _P, _P, _F, _P, _P, _I, _I, _P, _I, _L, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "llmp_capped_attention": [_P, _L, _P, _I, _P, _I, _P, _P, _P, _P, _P, _L, _I, _P, _L, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
+    "llmp_capped_attention_mma": [_P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F,
+                                  _I, _I, _I, _P, _P, _I, _P],
     "llmp_selective_scan": [_P, _L, _P, _L, _P, _P, _P, _L, _P, _P, _P, _L, _P, _L, _L, _P, _P, _P, _P, _I, _L, _I, _I, _I, _P],
     "llmp_add_rmsnorm_multi": [_P, _P, _I, _P, _I, _P, _I, _P, _I, _I, _F, _P, _I, _L, _L, _P, _I, _I, _P],
     "llmp_gated_act": [_P, _I, _L, _P, _I, _L, _I, _I, _P],
     "llmp_sigmoid_gate": [_P, _P, _L, _P, _I, _L, _I, _P],
     "llmp_convert_rows": [_P, _L, _P, _I, _L, _I, _P],
-    "llmp_route_topk": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P],
+    "llmp_route_topk": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P, _P],
     "llmp_expert_grouped": [_P, _P, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "llmp_expert_rows": [_P, _P, _P, _I, _P, _P, _F, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "llmp_add_layernorm": [_P, _P, _I, _P, _I, _P, _P, _I, _F, _P, _I, _I, _I, _P, _P],
@@ -94,6 +97,10 @@ _SIGNATURES = {
     "llmp_sig_qkv_post": [_P, _L, _P, _I, _P, _P, _I, _P, _I, _L, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "llmp_sigmoid_attention": [_P, _L, _P, _I, _P, _I, _P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "llmp_sigmoid_attention_mma": [_P, _L, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
+    "llmp_wkv_shift": [_P, _P, _P, _L, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "llmp_wkv_decay": [_P, _L, _P, _P, _P, _I, _I, _I, _P],
+    "llmp_wkv_scan": [_P, _P, _P, _L, _P, _L, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _P],
+    "llmp_wkv_gate": [_P, _L, _P, _L, _P, _P, _I, _L, _I, _I, _I, _F, _P],
     "llmp_xielu": [_P, _P, _I, _F, _F, _P, _I, _L, _I, _P],
     "llmp_scaled_sum": [_P, _F, _P, _F, _P, _L, _P],
 }
@@ -205,6 +212,26 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: 
           "embedding output must be float32 [tokens, hidden]")
     _call("llmp_embedding", _ptr(ids), _ptr(table), dtype_code(table.dtype), _ptr(out), ids.numel(),
           table.shape[1], table.shape[0], float(scale), _stream())
+    return out
+
+
+def embedding_bigram(ids: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor,
+                     positions: torch.Tensor, token_request: torch.Tensor, state: torch.Tensor, mul_prev: int, mul_cur: int,
+                     buckets: int, out: torch.Tensor) -> torch.Tensor:
+    """out[n, :] = table[ids[n], :] + bigram[row, :], row = (previous id * mul_prev + ids[n] * mul_cur) mod buckets, or
+    ``buckets`` for a request's first token. ``state`` int32 [slots, 2]: the last token of a request, two copies that take
+    turns by the parity of its position."""
+    for t, name in ((ids, "ids"), (q_start, "q_start"), (slots, "slots"), (positions, "positions"), (token_request, "token_request"),
+                    (state, "state")):
+        _i32(t, name)
+    _need(table.dim() == 2 and table.is_contiguous() and bigram.is_contiguous() and bigram.dtype == table.dtype and
+          bigram.shape == (buckets + 1, table.shape[1]), "the bigram table must be [buckets + 1, hidden] of the table's type")
+    _need(state.dim() == 2 and state.shape[1] == 2 and state.is_contiguous(), "the bigram state must be int32 [slots, 2]")
+    _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape == (ids.numel(), table.shape[1]),
+          "embedding output must be float32 [tokens, hidden]")
+    _call("llmp_embedding_bigram", _ptr(ids), _ptr(table), _ptr(bigram), dtype_code(table.dtype), _ptr(q_start), _ptr(slots),
+          _ptr(positions), _ptr(token_request), _ptr(state), int(mul_prev), int(mul_cur), int(buckets), _ptr(out), ids.numel(),
+          table.shape[1], table.shape[0], _stream())
     return out
 
 
@@ -790,7 +817,7 @@ def add_norm_mix(residual: torch.Tensor, *, delta: Optional[torch.Tensor] = None
     """The residual stream's norm kernel in its general form, per row r (``rows`` selects rows and leaves the stream as it is):
     y = delta[r], normed by (delta_offset + delta_weight) if that is given; x = residual[r] + y; with ``history``
     [slots, tokens, width]: history[index][r] = x and x = sum_{j <= index} mix[j] history[j][r]; residual[r] = x;
-    out = rms_norm(x) * (offset + weight) if ``out`` is given."""
+    out = rms_norm(x) * (offset + weight) if ``out`` is given (x itself without a weight)."""
     T, H = residual.shape
     _need(residual.dtype == torch.float32 and residual.is_contiguous(), "residual must be a contiguous float32 matrix")
     M = rows.numel() if rows is not None else T
@@ -804,7 +831,7 @@ def add_norm_mix(residual: torch.Tensor, *, delta: Optional[torch.Tensor] = None
         _need(mix is not None and mix.dtype == torch.float32 and mix.is_contiguous() and mix.numel() >= index + 1,
               "mixing weights must be float32, one per result so far")
     if out is not None:
-        _need(out.is_contiguous() and out.shape == (M, H) and weight is not None and weight.numel() == H and weight.is_contiguous(),
+        _need(out.is_contiguous() and out.shape == (M, H) and (weight is None or (weight.numel() == H and weight.is_contiguous())),
               "norm output or weight has the wrong shape")
     if rows is not None:
         _i32(rows, "rows")
@@ -916,11 +943,16 @@ def _sink(sink: Optional[torch.Tensor], heads: int) -> None:
           "a sink is one float32 number per head")
 
 
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1, "chosen_softmax": 2}
+
+
 def route_topk(h: torch.Tensor, w_router: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor, *,
-               softmax: bool = False, correction: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+               softmax: bool = False, score: Optional[str] = None, bias: Optional[torch.Tensor] = None,
+               correction: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """ids[n, :], weights[n, :] = the ``top`` router outputs with the largest score (+ ``correction``, if given) and their
-    scores without the correction; float32 logits. The score is sigmoid(logit), or with ``softmax`` the softmax over all
-    router outputs. With ``gate`` (float32 [tokens]) the matrix has one row more than router outputs, and
+    scores without the correction; float32 logits (+ ``bias``). The score is sigmoid(logit), or the softmax over all router
+    outputs (``score`` "softmax", or ``softmax`` set); "chosen_softmax": the ``top`` largest logits, and the softmax over
+    those. With ``gate`` (float32 [tokens]) the matrix has one row more than router outputs, and
     gate[n] = sigmoid(that row . h[n])."""
     N, Hd = h.shape
     E = w_router.shape[0] - (1 if gate is not None else 0)
@@ -928,29 +960,33 @@ def route_topk(h: torch.Tensor, w_router: torch.Tensor, top: int, ids: torch.Ten
           "the router matrix must be float32 [experts, width]")
     _need(ids.dtype == torch.int32 and ids.is_contiguous() and ids.shape == (N, top) and weights.dtype == torch.float32 and
           weights.is_contiguous() and weights.shape == (N, top), "route_topk outputs must be int32 and float32 [tokens, top]")
+    if bias is not None:
+        _need(bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == E, "the router's bias must be float32 [router outputs]")
     if correction is not None:
         _need(correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == E,
               "the router's correction must be float32 [router outputs]")
     if gate is not None:
         _need(gate.dtype == torch.float32 and gate.is_contiguous() and gate.numel() == N, "the gate must be float32 [tokens]")
     _call("llmp_route_topk", _ptr(h), dtype_code(h.dtype), _ptr(w_router), int(top), _ptr(ids), _ptr(weights), N, Hd, E,
-          1 if softmax else 0, _ptr(correction), _ptr(gate), _stream())
+          ROUTER_SCORES[score or ("softmax" if softmax else "sigmoid")], _ptr(bias), _ptr(correction), _ptr(gate), _stream())
 
 
-EXPERT_FORMS = {"clamped": 0, "silu": 1}     # csrc/routed_experts.cu: expert_act
+EXPERT_FORMS = {"clamped": 0, "silu": 1, "relu_squared": 2}     # csrc/routed_experts.cu: expert_act
+UNGATED_EXPERT_FORMS = ("relu_squared",)                        # their first matrix is [experts, ff, width]
 
 
 def expert_rows(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
                 limit: float, out: torch.Tensor, form: str = "clamped") -> torch.Tensor:
     """out[n] = sum_k Wd[e] act(Wg[e] h[n], Wu[e] h[n], weights[n, k]) with e = ids[n, k], float32; ``form`` names the
     activation and where the weight enters (``EXPERT_FORMS``); an id from the number of experts on adds weights[n, k] h[n].
-    ``w_gate_up`` [experts, 2 ff, width] (gate rows, then up rows), ``w_down`` [experts, width, ff]. Reads an expert once
+    ``w_gate_up`` [experts, 2 ff, width] (gate rows, then up rows; [experts, ff, width] for a form without a gate), ``w_down``
+    [experts, width, ff]. Reads an expert once
     per token that chose it: for the few rows of a decode step."""
     N, Hd = h.shape
-    E, two_f, _ = w_gate_up.shape
-    F = two_f // 2
+    E, rows_f, _ = w_gate_up.shape
+    F = rows_f if form in UNGATED_EXPERT_FORMS else rows_f // 2
     top = ids.shape[1]
-    _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and w_gate_up.shape == (E, 2 * F, Hd) and
+    _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and rows_f == (F if form in UNGATED_EXPERT_FORMS else 2 * F) and w_gate_up.shape[2] == Hd and
           w_down.shape == (E, Hd, F) and h.dtype == w_gate_up.dtype == w_down.dtype, "expert matrices have the wrong layout")
     _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape == (N, Hd), "expert output must be float32 [tokens, width]")
     y = torch.empty((N * top, F), dtype=h.dtype, device=h.device)
@@ -976,10 +1012,10 @@ def expert_grouped(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tenso
     """``expert_rows`` for many rows (bfloat16): the pairs are sorted by expert on the device and the experts' products
     run as grouped tensor-core products that read an expert's rows once per 64 pairs."""
     N, Hd = h.shape
-    E, two_f, _ = w_gate_up.shape
-    F = two_f // 2
+    E, rows_f, _ = w_gate_up.shape
+    F = rows_f if form in UNGATED_EXPERT_FORMS else rows_f // 2
     top = ids.shape[1]
-    _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and w_gate_up.shape == (E, 2 * F, Hd) and
+    _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and rows_f == (F if form in UNGATED_EXPERT_FORMS else 2 * F) and w_gate_up.shape[2] == Hd and
           w_down.shape == (E, Hd, F) and h.dtype == w_gate_up.dtype == w_down.dtype == torch.bfloat16, "expert matrices have the wrong layout")
     _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape == (N, Hd), "expert output must be float32 [tokens, width]")
     fn = library().llmp_expert_grouped_rows
@@ -1474,15 +1510,52 @@ def capped_qkv_post(qkv: torch.Tensor, bias: Optional[torch.Tensor], value_norm_
     return q_out
 
 
+def capped_rows_post(proj: torch.Tensor, q_weight: torch.Tensor, k_weight: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor],
+                     sin: Optional[torch.Tensor], rotary_dim: int, interleaved: bool, q_out: torch.Tensor,
+                     slot_mapping: Optional[torch.Tensor], pages: Optional[torch.Tensor], v_at: int, heads: int, kv_heads: int, dim: int,
+                     vdim: int) -> torch.Tensor:
+    """After the float32 product [q | k | ..] (csrc/capped_attention.cu): the whole rows of q and of k divided by their root mean
+    square times ``q_weight`` [heads dim] and ``k_weight`` [kv_heads dim] (float32), the first ``rotary_dim`` entries of every head
+    rotated (``interleaved``: entry 2i with 2i + 1), queries to ``q_out``, the token's [k | v] rows to its page slot with the
+    values as projected in the columns from ``v_at`` on. ``pages`` None: the queries alone (``proj`` may hold no k)."""
+    N = proj.shape[0]
+    nq, nk = heads * dim, kv_heads * dim
+    _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= nq, "capped_rows_post takes the float32 product [q | k | ..]")
+    for w, n in ((q_weight, nq), (k_weight if pages is not None else None, nk)):
+        _need(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == n), "capped_rows_post: row norms take float32 weights")
+    _need(q_out.shape == (N, nq) and q_out.stride(1) == 1, "capped_rows_post: the query output has the wrong shape")
+    for t in (cos, sin):
+        _need((t is None) == (rotary_dim == 0) and (t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == (N, rotary_dim // 2))),
+              "capped_rows_post: rotation tables must be float32 [tokens, rotary_dim / 2]")
+    page_size = 0
+    if pages is not None:
+        _need(k_weight is not None and proj.shape[1] >= max(nq + nk, v_at + kv_heads * vdim), "capped_rows_post: keys and values are missing from the product")
+        _need(slot_mapping is not None and pages.dim() == 4 and pages.is_contiguous() and pages.shape[1] == kv_heads and
+              pages.shape[3] == dim + vdim and pages.dtype == q_out.dtype, "capped_rows_post: pages must be [pages, kv_heads, page_size, dim + vdim] of the queries' type")
+        _i32(slot_mapping, "slot_mapping")
+        page_size = pages.shape[2]
+    _call("llmp_capped_rows_post", _ptr(proj), proj.stride(0), _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(cos), _ptr(sin), int(rotary_dim),
+          1 if interleaved else 0, _ptr(q_out), dtype_code(q_out.dtype), q_out.stride(0), _ptr(slot_mapping) if pages is not None else None,
+          _ptr(pages), page_size, int(v_at), N, heads, kv_heads, dim, vdim, _stream())
+    return q_out
+
+
+def _capped_gate(gate: Optional[torch.Tensor], tokens: int, num_heads: int, vdim: int) -> bool:
+    """Whether a gate is one number per head (else per channel)."""
+    _need(gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == tokens and
+                           gate.shape[1] in (num_heads, num_heads * vdim)), "the gate must be float32 [tokens, heads vdim] or [tokens, heads]")
+    return gate is not None and vdim > 1 and gate.shape[1] == num_heads
+
+
 def capped_attention(q: torch.Tensor, pages: torch.Tensor, tables: torch.Tensor, token_request: torch.Tensor, positions: torch.Tensor,
                      out: torch.Tensor, num_heads: int, num_kv_heads: int, dim: int, vdim: int, window: int, keep_first: int,
                      scale: float, softcap: float, slopes: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
-                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     gate: Optional[torch.Tensor] = None, chunk: int = 0) -> torch.Tensor:
     """Softmax attention of rows (token, head), any sizes, float32 or bfloat16 (csrc/capped_attention.cu): ``q`` [tokens, heads
     dim], ``pages`` [pages, kv_heads, page_size, dim + vdim], ``out`` [tokens, heads vdim]. A token sees the ``window`` keys up
-    to itself (0: all) and the first ``keep_first`` keys; a score is capped (``softcap`` > 0) and loses ``slopes[h]`` times the
-    distance; exp(``sink[h]``) joins the denominator; the result is multiplied by sigmoid(``gate``) (float32 [tokens, heads vdim],
-    a view)."""
+    to itself (0: all; with ``chunk`` only those of its own chunk) and the first ``keep_first`` keys; a score is capped (``softcap`` > 0) and loses ``slopes[h]`` times the
+    distance; exp(``sink[h]``) joins the denominator; the result is multiplied by sigmoid(``gate``) (float32 [tokens, heads vdim] or
+    [tokens, heads], a view)."""
     N = q.shape[0]
     _need(q.stride(1) == 1 and q.shape[1] == num_heads * dim and out.shape == (N, num_heads * vdim) and out.stride(1) == 1,
           "capped attention shapes do not match")
@@ -1490,14 +1563,17 @@ def capped_attention(q: torch.Tensor, pages: torch.Tensor, tables: torch.Tensor,
     _need(pages.is_contiguous() and pages.dim() == 4 and pages.shape[1] == num_kv_heads and pages.shape[3] == dim + vdim,
           "capped attention pages have the wrong layout")
     _sink(sink, num_heads); _sink(slopes, num_heads)
-    _need(gate is None or (gate.dtype == torch.float32 and gate.shape == (N, num_heads * vdim) and gate.stride(1) == 1),
-          "the gate must be float32 [tokens, heads vdim]")
+    gate_heads = _capped_gate(gate, N, num_heads, vdim)
     _i32(tables, "tables"); _i32(token_request, "token_request"); _i32(positions, "positions")
     _call("llmp_capped_attention", _ptr(q), q.stride(0), _ptr(pages), dtype_code(pages.dtype), _ptr(tables), tables.shape[1],
           _ptr(token_request), _ptr(positions), _ptr(slopes), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0,
-          _ptr(out), out.stride(0), N, num_heads, num_kv_heads, dim, vdim, pages.shape[2], int(window), int(keep_first),
-          float(scale), float(softcap), _stream())
+          1 if gate_heads else 0, _ptr(out), out.stride(0), N, num_heads, num_kv_heads, dim, vdim, pages.shape[2], int(window),
+          int(keep_first), int(chunk), float(scale), float(softcap), _stream())
     return out
+
+
+CAPPED_TILE_KEYS = 64                # csrc/capped_attention_mma.cu: keys of a tile
+CAPPED_SEGMENT_KEYS = 256            # keys of a segment (a multiple of the tile)
 
 
 def capped_mma_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:
@@ -1520,10 +1596,13 @@ def capped_mma_tokens_per_tile(num_heads: int, num_kv_heads: int) -> int:
 def capped_attention_mma(q: torch.Tensor, pages: torch.Tensor, tables: torch.Tensor, q_start: torch.Tensor, ctx_len: torch.Tensor,
                          tile_req: torch.Tensor, tile_tok0: torch.Tensor, out: torch.Tensor, num_heads: int, num_kv_heads: int, dim: int,
                          vdim: int, window: int, keep_first: int, scale: float, softcap: float, slopes: Optional[torch.Tensor] = None,
-                         sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, split: bool = False) -> torch.Tensor:
+                         sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, split: bool = False, chunk: int = 0,
+                         segments: int = 0) -> torch.Tensor:
     """``capped_attention`` on the tensor cores for bfloat16 (csrc/capped_attention_mma.cu). ``tile_req``/``tile_tok0``: the work
     list (request and first token of every tile of ``capped_mma_tokens_per_tile`` tokens). ``split``: every tile is one token,
-    and the four warps of a block share its keys."""
+    and the four warps of a block share its keys; ``segments`` > 0 then cuts the keys of a row into that many runs of
+    ``CAPPED_SEGMENT_KEYS`` with blocks of their own, whose sums the block that ends last adds up (it must cover the most keys a
+    token sees, rounded up to whole tiles at both ends)."""
     N = q.shape[0]
     _need(q.dtype == torch.bfloat16 and pages.dtype == torch.bfloat16 and out.dtype == torch.bfloat16, "capped_attention_mma takes bfloat16")
     _need(q.stride(1) == 1 and q.shape[1] == num_heads * dim and out.shape == (N, num_heads * vdim) and out.stride(1) == 1,
@@ -1531,15 +1610,23 @@ def capped_attention_mma(q: torch.Tensor, pages: torch.Tensor, tables: torch.Ten
     _need(pages.is_contiguous() and pages.dim() == 4 and pages.shape[1] == num_kv_heads and pages.shape[3] == dim + vdim,
           "capped attention pages have the wrong layout")
     _sink(sink, num_heads); _sink(slopes, num_heads)
-    _need(gate is None or (gate.dtype == torch.float32 and gate.shape == (N, num_heads * vdim) and gate.stride(1) == 1),
-          "the gate must be float32 [tokens, heads vdim]")
+    gate_heads = _capped_gate(gate, N, num_heads, vdim)
     for t, name in ((tables, "tables"), (q_start, "q_start"), (ctx_len, "ctx_len"), (tile_req, "tile_req"), (tile_tok0, "tile_tok0")):
         _i32(t, name)
     _need(not split or tile_req.numel() == N, "warps share a tile's keys only in steps of one token a request")
+    scratch = counters = None
+    if split:
+        # at most one counter per (tile, kv head, chunk of heads); asked for in every such step, so that they exist before a step
+        # is captured whose eager run needed no segments
+        counters = attention_counters(q.device, tile_req.numel() * num_heads)
+    if segments > 0:
+        _need(split, "capped_attention_mma: segments are for steps of one token a request")
+        scratch = torch.empty(segments * N * num_heads * (vdim + 2), dtype=torch.float32, device=q.device)
     _call("llmp_capped_attention_mma", _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(pages), _ptr(tables), tables.shape[1],
           _ptr(q_start), _ptr(ctx_len), _ptr(tile_req), _ptr(tile_tok0), tile_req.numel(), _ptr(slopes), _ptr(sink), _ptr(gate),
-          gate.stride(0) if gate is not None else 0, num_heads, num_kv_heads, dim, vdim, pages.shape[2], int(window), int(keep_first),
-          float(scale), float(softcap), 1 if split else 0, _stream())
+          gate.stride(0) if gate is not None else 0, 1 if gate_heads else 0, num_heads, num_kv_heads, dim, vdim, pages.shape[2],
+          int(window), int(keep_first), int(chunk), float(scale), float(softcap), 1 if split else 0, int(segments),
+          CAPPED_SEGMENT_KEYS if segments > 0 else 0, _ptr(scratch), _ptr(counters), N, _stream())
     return out
 
 
@@ -1619,4 +1706,75 @@ def convert_rows(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     """Float32 rows (a view with a dense last axis) as dense rows of ``out``'s type."""
     _need(x.dtype == torch.float32 and x.dim() == 2 and x.stride(1) == 1 and out.is_contiguous() and out.shape == x.shape, "convert_rows shapes do not match")
     _call("llmp_convert_rows", _ptr(x), x.stride(0), _ptr(out), dtype_code(out.dtype), x.shape[0], x.shape[1], _stream())
+    return out
+
+
+WKV_MAX_DIM = 256
+
+
+def wkv_state_entries(heads: int, dim: int) -> int:
+    """Entries of one copy of the wkv recurrence's state as csrc/wkv.cu keeps it: per head and block of 16 value columns, two
+    columns of ``rows`` rows for each of 16 lanes of 8 half-warps (16 ``rows`` >= dim, a power of two)."""
+    rows = 1
+    while 16 * rows < dim:
+        rows *= 2
+    return heads * -(-dim // 16) * 2 * rows * 128
+
+
+def wkv_shift(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, state_offset: int, q_start: torch.Tensor, slots: torch.Tensor,
+              positions: torch.Tensor, token_request: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out[s, t] = x_t + (x_(t-1) - x_t) mu[s] for float32 rows ``x`` [tokens, width] (zeros before a request's first token),
+    ``mu`` float32 [k, width], ``out`` [k, tokens, width] in float32 or bfloat16. The state piece holds two copies of a row."""
+    N, D = x.shape
+    k = mu.shape[0]
+    _need(x.dtype == torch.float32 and x.is_contiguous() and mu.dtype == torch.float32 and mu.is_contiguous() and mu.shape == (k, D),
+          "wkv_shift takes float32 rows and mixes")
+    _need(out.is_contiguous() and out.shape == (k, N, D), "wkv_shift: the output must be [mixes, tokens, width]")
+    for t, name in ((q_start, "q_start"), (slots, "slots"), (positions, "positions"), (token_request, "token_request")):
+        _i32(t, name)
+    ptr, slot_stride, half = _state_views(state, state_offset, D, "wkv_shift")
+    _call("llmp_wkv_shift", _ptr(x), _ptr(mu), ptr, slot_stride, half, _ptr(q_start), _ptr(slots), _ptr(positions), _ptr(token_request),
+          _ptr(out), dtype_code(out.dtype), N, D, k, _stream())
+    return out
+
+
+def wkv_decay(low: torch.Tensor, w2t: torch.Tensor, w0: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out = exp(-exp(tanh(low) @ w2t + w0)): ``low`` float32 [tokens, rank], ``w2t`` float32 [rank, channels], ``out`` float32
+    [tokens, channels]."""
+    N, rank = low.shape
+    C = w0.numel()
+    _need(low.dtype == torch.float32 and low.stride(1) == 1 and w2t.dtype == torch.float32 and w2t.is_contiguous() and
+          w2t.shape == (rank, C) and w0.dtype == torch.float32 and w0.is_contiguous(), "wkv_decay takes float32 operands")
+    _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape == (N, C), "wkv_decay: the output must be float32 [tokens, channels]")
+    _call("llmp_wkv_decay", _ptr(low), low.stride(0), _ptr(w2t), _ptr(w0), _ptr(out), N, C, rank, _stream())
+    return out
+
+
+def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, bonus: torch.Tensor, state: torch.Tensor,
+             state_offset: int, q_start: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, heads: int,
+             dim: int) -> torch.Tensor:
+    """The wkv recurrence over the step's tokens, request by request (csrc/wkv.cu): ``r``, ``k``, ``v``, ``decay``, ``out`` float32
+    [tokens, heads dim], ``bonus`` float32 [heads, dim]. The state piece holds two copies of ``wkv_state_entries`` floats."""
+    N = r.shape[0]
+    for t, name in ((r, "r"), (k, "k"), (v, "v"), (decay, "decay"), (out, "out")):
+        _need(t.dtype == torch.float32 and t.stride(1) == 1 and t.shape == (N, heads * dim), f"wkv_scan: {name} must be float32 [tokens, heads dim]")
+    _need(r.stride(0) == k.stride(0) == v.stride(0), "wkv_scan: r, k and v have one row stride")
+    _need(bonus.dtype == torch.float32 and bonus.is_contiguous() and bonus.shape == (heads, dim), "wkv_scan: the bonus must be float32 [heads, dim]")
+    for t, name in ((q_start, "q_start"), (slots, "slots"), (positions, "positions")):
+        _i32(t, name)
+    ptr, slot_stride, half = _state_views(state, state_offset, wkv_state_entries(heads, dim), "wkv_scan")
+    _call("llmp_wkv_scan", _ptr(r), _ptr(k), _ptr(v), r.stride(0), _ptr(decay), decay.stride(0), _ptr(bonus), ptr, slot_stride, half,
+          _ptr(q_start), _ptr(slots), _ptr(positions), _ptr(out), out.stride(0), slots.numel(), heads, dim, _stream())
+    return out
+
+
+def wkv_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, heads: int, dim: int, eps: float) -> torch.Tensor:
+    """out = rms(o per head) * weight * silu(gate): float32 rows ``o`` and ``gate`` [tokens, heads dim], ``weight`` float32 [heads dim]."""
+    N = o.shape[0]
+    for t, name in ((o, "o"), (gate, "gate")):
+        _need(t.dtype == torch.float32 and t.stride(1) == 1 and t.shape == (N, heads * dim), f"wkv_gate: {name} must be float32 [tokens, heads dim]")
+    _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == heads * dim, "wkv_gate: the weight has the wrong size")
+    _need(out.shape == (N, heads * dim) and out.stride(1) == 1, "wkv_gate: the output has the wrong shape")
+    _call("llmp_wkv_gate", _ptr(o), o.stride(0), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(out), dtype_code(out.dtype), out.stride(0),
+          N, heads, dim, float(eps), _stream())
     return out

@@ -126,7 +126,8 @@ class ResidualStream:
 
     def fold(self, weight: Optional[torch.Tensor] = None, eps: float = 0.0, out: Optional[torch.Tensor] = None,
              rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-        """Everything pending in one kernel, and the RMS norm of the result by ``weight`` into ``out`` if given. With
+        """Everything pending in one kernel, and the RMS norm of the result by ``weight`` (without one: the result itself)
+        into ``out`` if given. With
         ``rows`` only those rows are computed and the stream stays as it is."""
         from ..ops import kernels
 
@@ -143,6 +144,17 @@ class ResidualStream:
         if rows is None:
             self._pending, self.pending_bias, self.pending_norm, self.pending_mix = None, None, None, None
         return out
+
+    def settled_rows(self, dtype: torch.dtype) -> torch.Tensor:
+        """The stream's rows themselves, everything pending added, for a sublayer that reads them without a norm: the
+        float32 residual or, for another type, a copy rounded once (by the kernel that does the adding)."""
+        from ..ops import kernels
+
+        out = torch.empty(self.residual.shape, dtype=dtype, device=self.residual.device) if dtype != torch.float32 else None
+        if self.pending is None and self.plain:
+            return kernels.convert_rows(self.residual, out) if out is not None else self.residual
+        self.fold(out=out)
+        return out if out is not None else self.residual
 
     def settle(self) -> torch.Tensor:
         """Add what is pending into the residual and return it: the whole state of the stream in one float32 tensor
@@ -244,8 +256,16 @@ class DepthMix(Part):
 
 
 class Embedding(Part):
+    def state_spec(self) -> Optional[StateSpec]:
+        """What the embedding carries from token to token of a request (None: nothing; it is called through ``forward``)."""
+        return None
+
     def forward(self, ctx) -> torch.Tensor:
         """float32 residual [tokens, hidden] of ctx.token_ids"""
+        raise NotImplementedError
+
+    def forward_with_state(self, ctx, state: torch.Tensor) -> torch.Tensor:
+        """The same for an embedding with a ``state_spec``: ``state`` is its tensor ``[slots, ...]``."""
         raise NotImplementedError
 
 

@@ -63,6 +63,30 @@ class SandwichNormResidualBlock(Block):
             stream.mix(self.depth_mix.weights, self.depth_mix.index)
 
 
+@register_block("output_norm_residual")
+class OutputNormResidualBlock(Block):
+    """A norm on each sublayer's output alone: ``x += norm_mixer(mixer(x))``, then ``x += norm_ff(feed_forward(x))`` if the
+    layer has a feed-forward; a sublayer reads the residual itself. A sublayer's output is left pending on the stream with
+    its norm; the kernel that norms and adds it also leaves the sum rounded to the compute type for the next reader. A part
+    with ``reads_float32`` gets the float32 residual instead (it may rely on it only until it returns)."""
+
+    NORMS = ("mixer_out", "feed_forward_out")
+
+    def needed_norms(self):
+        return self.NORMS if self.feed_forward is not None else ("mixer_out",)
+
+    @staticmethod
+    def _rows(stream: ResidualStream, ctx, part) -> torch.Tensor:
+        return stream.settled_rows(torch.float32 if getattr(part, "reads_float32", False) else ctx.dtype)
+
+    def forward(self, stream: ResidualStream, ctx, cache: LayerCache) -> None:
+        out, bias = self.mixer.forward(self._rows(stream, ctx, self.mixer), ctx, cache)
+        stream.add(out, bias, norm=self.norms["mixer_out"])
+        if self.feed_forward is not None:
+            out, bias = self.feed_forward.forward(self._rows(stream, ctx, self.feed_forward), ctx)
+            stream.add(out, bias, norm=self.norms["feed_forward_out"])
+
+
 @register_block("parallel_residual")
 class ParallelResidualBlock(Block):
     """Both sublayers read the same residual: ``x += mixer(norm(x)) + feed_forward(norm(x))`` (a layer without a

@@ -8,6 +8,7 @@ from typing import Dict, Optional
 
 import torch
 
+from ..cache.spec import StateSpec
 from ..ops import kernels
 from ..ops.linear import linear
 from ..weights.source import ParamSpec
@@ -62,6 +63,41 @@ class NormedTokenEmbedding(TokenEmbedding):
         out = torch.empty((ctx.num_tokens, self.hidden_size), dtype=torch.float32, device=ctx.device)
         kernels.embedding_norm(ctx.token_ids, self.weight, self.norm_weight, 0.0, self.eps, out)
         return out
+
+
+@register_embedding("bigram_token_embedding")
+class BigramTokenEmbedding(TokenEmbedding):
+    """The token's row plus a row of a second table that the previous and the current token choose together:
+    ``(previous * mul_prev + current * mul_cur) mod buckets``, and row ``buckets`` (the table's last) for a request's first
+    token. The sum is float32. The previous token of a step's first token is carried on the device, in the request's
+    slot: two copies that take turns by the parity of the last position written, so that a replayed decode step (whose
+    token the host may not have seen yet) reads what it did not write."""
+
+    def __init__(self, prefix: str, vocab_size: int, hidden_size: int, buckets: int, mul_prev: int, mul_cur: int,
+                 name: Optional[str] = None, table_name: Optional[str] = None):
+        super().__init__(prefix, vocab_size, hidden_size, name)
+        self.buckets, self.mul_prev, self.mul_cur = int(buckets), int(mul_prev), int(mul_cur)
+        if self.buckets <= 0:
+            raise ValueError(f"a bigram table needs buckets, got {buckets}")
+        self.table_name = table_name or f"{prefix}.bigram"
+        self.bigram: Optional[torch.Tensor] = None
+
+    def state_spec(self) -> StateSpec:
+        return StateSpec((2,), torch.int32)
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        specs = super().param_specs()
+        specs[self.table_name] = ParamSpec((self.buckets + 1, self.hidden_size))
+        return specs
+
+    def load(self, get: TensorGetter) -> None:
+        super().load(get)
+        self.bigram = get(self.table_name, "matrix").contiguous()
+
+    def forward_with_state(self, ctx, state: torch.Tensor) -> torch.Tensor:
+        out = torch.empty((ctx.num_tokens, self.hidden_size), dtype=torch.float32, device=ctx.device)
+        return kernels.embedding_bigram(ctx.token_ids, self.weight, self.bigram, ctx.q_start, ctx.slots, ctx.positions,
+                                        ctx.token_request, state, self.mul_prev, self.mul_cur, self.buckets, out)
 
 
 @register_head("linear_head")

@@ -3,21 +3,23 @@
 With h the feed-forward's input, E experts with matrices, ``identity`` further router outputs without any, and ``top``
 choices per token::
 
-    z = Wr h                                  router logits, float32; one per expert and identity expert
+    z = Wr h (+ b)                            router logits, float32; one per expert and identity expert (``router_bias``: b)
     s = sigmoid(z)  or  softmax(z)            ``score``: each logit alone, or over all router outputs
     chosen = the top outputs by s (+ correction, a stored vector, if the router has one)
+                                              ``score`` "chosen_softmax": the top outputs by z, s = softmax over those alone
     an expert's weight w is its s (without the correction, not renormalised)
     expert_e(v), ``form`` "clamped": g = min(Wg_e v, limit), u = clamp(Wu_e v, -limit, limit), y = g sigmoid(1.702 g) (u + 1),
                                      Wd_e y, and the weight scales the expert's input: out += expert_e(w h)
                  ``form`` "silu":    Wd_e (silu(Wg_e v) (Wu_e v)), and the weight scales its output: out += w expert_e(h)
+                 ``form`` "relu_squared":  Wd_e max(Wu_e v, 0)^2 without a gate, the weight on its output as well
     an identity expert adds w h
     ``shared_size``: one more expert of the "silu" form that every token uses, added times sigmoid(w_sg . h)
 
 The weight never makes a scaled copy: on the input side ``Wg_e (w h) = w (Wg_e h)`` puts it on the float32 sums of the
 first two products, on the output side ``w (Wd_e y) = Wd_e (w y)`` puts it on the float32 activation. Routing happens on
 the device (``csrc/routed_experts.cu``): nothing of a step depends on the host seeing the choices, so the part can be
-captured in a CUDA graph. The experts' matrices are stacked: ``[E, 2 ff, hidden]`` (gate rows, then up rows) and
-``[E, hidden, ff]``. The shared expert's gate is one more row of the float32 router matrix; its products are the
+captured in a CUDA graph. The experts' matrices are stacked: ``[E, 2 ff, hidden]`` (gate rows, then up rows; ``[E, ff,
+hidden]`` for a form without a gate) and ``[E, hidden, ff]``. The shared expert's gate is one more row of the float32 router matrix; its products are the
 engine's ``linear`` and fused gate/up kernels."""
 
 from __future__ import annotations
@@ -39,11 +41,13 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, num_experts: int, top: int, limit: float = 0.0,
                  score: str = "sigmoid", form: str = "clamped", identity: int = 0, correction: bool = False,
-                 shared_size: Optional[int] = None):
+                 shared_size: Optional[int] = None, router_bias: bool = False):
         if not 0 < top <= num_experts + identity:
             raise ValueError(f"a token cannot use {top} of {num_experts + identity} experts")
-        if score not in ("sigmoid", "softmax"):
-            raise ValueError(f"router scores are 'sigmoid' or 'softmax', not {score!r}")
+        if score not in kernels.ROUTER_SCORES:
+            raise ValueError(f"router scores are one of {sorted(kernels.ROUTER_SCORES)}, not {score!r}")
+        if score == "chosen_softmax" and correction:
+            raise ValueError("a softmax over the chosen logits takes them as they are: no correction")
         if form not in kernels.EXPERT_FORMS:
             raise ValueError(f"unknown expert form {form!r}; known: {sorted(kernels.EXPERT_FORMS)}")
         if num_experts < 1 or identity < 0:
@@ -52,6 +56,8 @@ class RoutedExperts(FeedForward):
         self.num_experts, self.top, self.limit = int(num_experts), int(top), float(limit)
         self.score, self.form, self.identity, self.correction = score, form, int(identity), bool(correction)
         self.shared_size = int(shared_size) if shared_size else None
+        self.router_bias, self.gated = bool(router_bias), form not in kernels.UNGATED_EXPERT_FORMS
+        self.b_router = None
         self.w_router = self.w_gate_up = self.w_down = self.router_correction = self.w_shared_gate_up = self.w_shared_down = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -60,8 +66,11 @@ class RoutedExperts(FeedForward):
         specs = {f"{p}.router": ParamSpec((outputs, H))}
         if self.correction:
             specs[f"{p}.correction"] = ParamSpec((outputs,), role="vector", init="small")
+        if self.router_bias:
+            specs[f"{p}.router.b"] = ParamSpec((outputs,), role="vector", init="small")
         for e in range(self.num_experts):
-            specs[f"{p}.e{e}.gate"] = ParamSpec((I, H))
+            if self.gated:
+                specs[f"{p}.e{e}.gate"] = ParamSpec((I, H))
             specs[f"{p}.e{e}.up"] = ParamSpec((I, H))
             specs[f"{p}.e{e}.down"] = ParamSpec((H, I))
         if self.shared_size:
@@ -80,7 +89,10 @@ class RoutedExperts(FeedForward):
         self.w_router = router.contiguous()
         if self.correction:
             self.router_correction = get(f"{p}.correction", "vector").float().contiguous()
-        self.w_gate_up = torch.stack([torch.cat([get(f"{p}.e{e}.gate", "matrix"), get(f"{p}.e{e}.up", "matrix")], dim=0)
+        if self.router_bias:
+            self.b_router = get(f"{p}.router.b", "vector").float().contiguous()
+        first = ("gate", "up") if self.gated else ("up",)
+        self.w_gate_up = torch.stack([torch.cat([get(f"{p}.e{e}.{n}", "matrix") for n in first], dim=0)
                                       for e in range(self.num_experts)]).contiguous()
         self.w_down = torch.stack([get(f"{p}.e{e}.down", "matrix") for e in range(self.num_experts)]).contiguous()
 
@@ -89,7 +101,7 @@ class RoutedExperts(FeedForward):
         ids = torch.empty((N, self.top), dtype=torch.int32, device=x.device)
         weights = torch.empty((N, self.top), dtype=torch.float32, device=x.device)
         gate = torch.empty((N,), dtype=torch.float32, device=x.device) if self.shared_size else None
-        kernels.route_topk(x, self.w_router, self.top, ids, weights, softmax=self.score == "softmax",
+        kernels.route_topk(x, self.w_router, self.top, ids, weights, score=self.score, bias=self.b_router,
                            correction=self.router_correction, gate=gate)
         out = torch.empty((N, self.hidden_size), dtype=torch.float32, device=x.device)
         kernels.routed_experts(x, self.w_gate_up, self.w_down, ids, weights, self.limit, out, self.form, self.identity)
