@@ -33,6 +33,8 @@ window beside a dense or routed-expert feed-forward on one layer norm).
 ``--compare tupidra [--size 1k|2k]`` does the same for the Tupidra decoder (a selective scan, capped window attention with
 kept first tokens, latent attention with query latents, sinks, gates and shared rows, each beside a gated GELU
 feed-forward behind norms and input filters of its own).
+``--compare zasudra [--size 1k|2k]`` does the same for the Zasudra decoder (chunked attention, a wkv recurrence, gated
+attention that may read another layer's keys, routed squared-ReLU experts).
 ``--compare nufolix [--size 1k|2k]`` does the same for the Nufolix decoder (a state-space mixer; sigmoid attention with
 mixed heads side by side with a gated delta rule; dense xIELU feed-forwards).
 
@@ -920,12 +922,73 @@ def tupidra_work(z, tokens, keys_per_token, decode, requests=1):
     return work
 
 
+# ``--compare zasudra``: the same two measurements for the Zasudra decoder: four layers (chunked attention with row norms and
+# values that are the keys; a wkv recurrence; causal attention with a gate per head; one more that reads the third layer's
+# keys and values), each with routed squared-ReLU experts, beside a Qwen3 dense decoder of the same width, depth and
+# vocabulary whose attention has the same heads of 128.
+ZASUDRA_SIZES = {
+    "1k": {"width": 1024, "heads": 8, "kv_heads": 4, "dim": 128, "chunk": 1024, "rot": 64, "heads2": 8, "kv_heads2": 4, "dim2": 128,
+           "wkv_heads": 16, "wkv_dim": 64, "experts": 16, "top": 4, "expert_ff": 1024, "buckets": 65521, "ff": 4096, "layers": 4,
+           "vocab": 32000, "qwen_heads": (8, 4)},
+    "2k": {"width": 2048, "heads": 16, "kv_heads": 8, "dim": 128, "chunk": 1024, "rot": 64, "heads2": 16, "kv_heads2": 8, "dim2": 128,
+           "wkv_heads": 32, "wkv_dim": 64, "experts": 32, "top": 4, "expert_ff": 1408, "buckets": 65521, "ff": 8192, "layers": 4,
+           "vocab": 32000, "qwen_heads": (16, 8)},
+}
+
+
+def zasudra_config(z):
+    mlp = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    causal = {"heads": z["heads2"], "kv_heads": z["kv_heads2"], "dim": z["dim2"], "vdim": z["dim2"], "scale": z["dim2"] ** -0.5}
+    kinds = [{"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"],
+                                             "scale": z["dim"] ** -0.5, "mask": {"size": z["chunk"]}, "rot": {"base": 10000.0, "dims": z["rot"]}}},
+             {"type": "wkv", "mixer": {"heads": z["wkv_heads"], "dim": z["wkv_dim"]}}, {"type": "attention_2", "mixer": causal}]
+    layers = [{**(kinds[i % 4] if i % 4 != 3 else {"type": "attention_2", "mixer": {**causal, "kv_from": i - 1}}), "mlp": mlp}
+              for i in range(z["layers"])]
+    return {"architecture": "Zasudra", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "logit_scale": 1.0, "embedding": {"bigram": {"buckets": z["buckets"], "mul_prev": 7919, "mul_cur": 104729}}, "layers": layers}
+
+
+def zasudra_work(z, tokens, keys_per_token, decode, requests=1):
+    """Closed-form work of the design's own kernel classes for one step: label -> (bytes, flops)."""
+    D, L = z["width"], z["layers"]
+    chunk_layers, wkv_layers, causal_layers = (L + 3) // 4, (L + 2) // 4, (L + 1) // 4 + L // 4
+    own_layers = (L + 1) // 4                                # causal layers with keys of their own
+    H, G, d = z["heads"], z["kv_heads"], z["dim"]
+    H2, G2, d2 = z["heads2"], z["kv_heads2"], z["dim2"]
+    C, hd = z["wkv_heads"] * z["wkv_dim"], z["wkv_dim"]
+    work = {}
+    # per sublayer the float32 output and the residual read, the residual written, a typed copy of it for the next reader
+    work["add_norm_mix"] = (2 * L * tokens * D * (4 + 4 + 4 + 2), 0.0)
+    work["wkv_shift"] = (wkv_layers * tokens * D * (4 + 5 * 2), 0.0)
+    work["wkv_decay"] = (wkv_layers * tokens * C * 4, 0.0)
+    work["wkv_scan"] = (wkv_layers * (tokens * C * (4 * 4 + 4) + requests * C * hd * 8), 0.0)
+    work["wkv_gate"] = (wkv_layers * tokens * C * (4 + 4 + 2), 0.0)
+    # float32 products in, queries and [k | v] rows out
+    work["capped_rows_post"] = (tokens * (chunk_layers * ((H + G) * d * (4 + 2) + G * d * 2) + causal_layers * H2 * d2 * 6 +
+                                          own_layers * 2 * G2 * d2 * 6), 0.0)
+    # a token's keys in its own chunk, on average over the step
+    if decode:
+        in_chunk = (CONTEXT - 1) % z["chunk"] + 1
+        work["capped_attention_mma"] = (tokens * 2 * 2 * (chunk_layers * in_chunk * G * d + causal_layers * keys_per_token * G2 * d2), 0.0)
+    else:
+        in_chunk = min(keys_per_token, (z["chunk"] + 1) / 2)
+        work["capped_attention_mma"] = (0.0, 4.0 * tokens * (chunk_layers * in_chunk * H * d + causal_layers * keys_per_token * H2 * d2))
+    pairs = tokens * z["top"]
+    if decode:
+        work["expert_rows"] = (L * pairs * 2 * z["expert_ff"] * D * 2, 0.0)
+    else:
+        work["expert_rows"] = (0.0, L * 2.0 * pairs * 2 * z["expert_ff"] * D)
+    work["expert_grouped"] = work["expert_rows"]
+    return work
+
+
 def run_compare(args):
     peak = peaks()
     sizes, config_of, work_of = {"zupilorn": (ZUPILORN_SIZES, zupilorn_config, zupilorn_work),
                                  "razelorn": (RAZELORN_SIZES, razelorn_config, razelorn_work),
                                  "nufolix": (NUFOLIX_SIZES, nufolix_config, lambda z, n, k, d: nufolix_work(z, n, k, d, args.batch if d else 1)),
-                                 "tupidra": (TUPIDRA_SIZES, tupidra_config, lambda z, n, k, d: tupidra_work(z, n, k, d, args.batch if d else 1))}[args.compare]
+                                 "tupidra": (TUPIDRA_SIZES, tupidra_config, lambda z, n, k, d: tupidra_work(z, n, k, d, args.batch if d else 1)),
+                                 "zasudra": (ZASUDRA_SIZES, zasudra_config, lambda z, n, k, d: zasudra_work(z, n, k, d, args.batch if d else 1))}[args.compare]
     z = sizes[args.size]
     clocks = ClockSampler()
     clocks.start()
@@ -1021,7 +1084,7 @@ def main() -> int:
     parser.add_argument("--lean", action="store_true", help="leave out the per-kernel breakdown, the page-size point, the plain "
                         "PyTorch baseline and the self-check")
     parser.add_argument("--page-size", type=int, default=PAGE_SIZE, help="tokens per page of the key/value cache")
-    parser.add_argument("--compare", default="", choices=("", "zupilorn", "razelorn", "nufolix", "tupidra"),
+    parser.add_argument("--compare", default="", choices=("", "zupilorn", "razelorn", "nufolix", "tupidra", "zasudra"),
                         help="instead of the headline: prefill and decode of this design at real layer sizes beside a Qwen3 dense "
                         "decoder of the same width and depth, with the time of every kernel class")
     parser.add_argument("--size", default="2k", choices=tuple(ZUPILORN_SIZES), help="with --compare: the layer sizes")

@@ -456,7 +456,7 @@ struct MapKeyHash {
 };
 
 // A [rows, K] bfloat16 row-major matrix with row pitch ld, read in boxes of box_rows x 64 elements.
-static int make_map(const void* ptr, long rows, long k, long ld, int box_rows, CUtensorMap* out) {
+int llmp_matrix_tensor_map(const void* ptr, long rows, long k, long ld, int box_rows, CUtensorMap* out) {
     static std::unordered_map<MapKey, CUtensorMap, MapKeyHash> cache;
     static std::mutex lock;
     const MapKey key{ptr, rows, k, ld, box_rows};
@@ -485,7 +485,7 @@ template <int BN, int STAGES, bool SWAP, typename TO>
 static int launch_tc(const void* A, long rows_a, long lda, const void* B, long rows_b, long ldb, TO* Y, int K, long ldy,
                      int* error_flag, cudaStream_t stream) {
     CUtensorMap map_a, map_b;
-    if (make_map(A, rows_a, K, lda, TC_BM, &map_a) || make_map(B, rows_b, K, ldb, BN, &map_b)) return 1;
+    if (llmp_matrix_tensor_map(A, rows_a, K, lda, TC_BM, &map_a) || llmp_matrix_tensor_map(B, rows_b, K, ldb, BN, &map_b)) return 1;
     constexpr size_t smem = (size_t)STAGES * (TC_BM * 128 + BN * 128) + 1024;
     auto kernel = gemm_tc_kernel<BN, STAGES, SWAP, TO>;
     LLMP_ALLOW_SMEM(kernel, smem);
@@ -527,7 +527,7 @@ template <int BN, int STAGES, typename TO>
 static int launch_tc_splitk(const void* A, long rows_a, long lda, const void* B, long rows_b, long ldb, TO* Y, int K,
                             long ldy, int* error_flag, cudaStream_t stream) {
     CUtensorMap map_a, map_b;
-    if (make_map(A, rows_a, K, lda, TC_BM, &map_a) || make_map(B, rows_b, K, ldb, BN, &map_b)) return 1;
+    if (llmp_matrix_tensor_map(A, rows_a, K, lda, TC_BM, &map_a) || llmp_matrix_tensor_map(B, rows_b, K, ldb, BN, &map_b)) return 1;
     constexpr size_t ring = (size_t)STAGES * (TC_BM * 128 + BN * 128);
     constexpr size_t smem = ring + 1024;
     auto kernel = gemm_tc_splitk_kernel<BN, STAGES, TO>;
@@ -561,7 +561,7 @@ template <int BN, int STAGES, typename TO>
 static int launch_tc_persistent(const void* A, long rows_a, long lda, const void* B, long rows_b, long ldb, TO* Y, int K,
                                 long ldy, int* error_flag, cudaStream_t stream) {
     CUtensorMap map_a, map_b;
-    if (make_map(A, rows_a, K, lda, TC_BM, &map_a) || make_map(B, rows_b, K, ldb, BN, &map_b)) return 1;
+    if (llmp_matrix_tensor_map(A, rows_a, K, lda, TC_BM, &map_a) || llmp_matrix_tensor_map(B, rows_b, K, ldb, BN, &map_b)) return 1;
     constexpr size_t smem = (size_t)STAGES * (TC_BM * 128 + BN * 128) + 1024;
     auto kernel = gemm_tc_persistent_kernel<BN, STAGES, TO>;
     LLMP_ALLOW_SMEM(kernel, smem);

@@ -15,16 +15,79 @@
 //   expert_down:     out[token] = sum over the token's choices, in their order, of Wd y (float32). A choice whose id is
 //                    not below the number of experts with matrices is an identity expert: it adds w h.
 // These kernels read an expert's rows once per token that chose it (a warp per output row): the form for the few
-// rows of a decode step. Steps with many rows sort their (token, choice) pairs by expert and take the grouped
-// product further down, which reads an expert's rows once per 64 pairs.
-#include "common.cuh"
+// rows of a decode step. Steps with more rows sort their (token, choice) pairs by expert: the grouped product further down
+// reads an expert's rows once per 64 pairs (mma.sync); many rows go to routed_experts_tc.cu (tcgen05).
+#include "routed_experts.cuh"
+
+// The choice of one token by one warp: `logits` [E (+ 1: the gate's)] in shared memory, overwritten; `score` [E] is scratch.
+__device__ __forceinline__ void route_choose(float* logits, float* score, int n, int top, int* __restrict__ ids, float* __restrict__ wts, int E,
+                                             int mode, const float* __restrict__ correction, float* __restrict__ gate, int lane) {
+    const bool softmax = mode == 1;
+    if (gate && lane == 0) gate[n] = 1.f / (1.f + expf(-logits[E]));
+    if (softmax) {
+        float mx = -INFINITY;
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, logits[e]);
+        mx = warp_max(mx);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) {
+            const float p = expf(logits[e] - mx);
+            score[e] = p;
+            sum += p;
+        }
+        sum = warp_sum(sum);
+        __syncwarp();
+        for (int e = lane; e < E; e += 32) {
+            const float p = score[e] / sum;
+            score[e] = p;
+            logits[e] = correction ? p + correction[e] : p;
+        }
+        __syncwarp();
+    } else if (correction) {
+        for (int e = lane; e < E; e += 32) {
+            score[e] = 1.f / (1.f + expf(-logits[e]));
+            logits[e] = score[e] + correction[e];
+        }
+        __syncwarp();
+    }
+    const bool by_score = softmax || correction;
+    float first = 0.f, total = 0.f;                      // mode 2: the largest logit, and the sum of the chosen exponentials
+    for (int k = 0; k < top; ++k) {
+        float best = -INFINITY;
+        int at = -1;
+        for (int e = lane; e < E; e += 32)
+            if (logits[e] > best) { best = logits[e]; at = e; }
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+            if (ob > best || (ob == best && oa >= 0 && (at < 0 || oa < at))) { best = ob; at = oa; }
+        }
+        if (at < 0) at = 0;                                  // logits that are not numbers: still an expert that exists
+        if (lane == 0) {
+            ids[(size_t)n * top + k] = at;
+            float w;
+            if (mode == 2) {
+                if (k == 0) first = best;
+                w = expf(best - first);
+                total += w;
+            } else {
+                w = by_score ? score[at] : 1.f / (1.f + expf(-best));
+            }
+            wts[(size_t)n * top + k] = w;
+            logits[at] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    if (mode == 2) {
+        total = __shfl_sync(0xffffffffu, total, 0);
+        for (int k = lane; k < top; k += 32) wts[(size_t)n * top + k] /= total;
+    }
+}
 
 __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const float* __restrict__ wr, int top, int* __restrict__ ids,
                                   float* __restrict__ wts, int Hd, int E, int mode, const float* __restrict__ bias,
                                   const float* __restrict__ correction, float* __restrict__ gate) {
     pdl_wait();                                    // what the kernels before wrote is complete
     pdl_trigger();
-    const bool softmax = mode == 1;
     extern __shared__ float route_smem[];
     float* logits = route_smem;                              // [E + 1]: logits, then what the choice goes by
     float* score = route_smem + E + 1;                       // [E]: softmax scores (softmax only)
@@ -50,65 +113,62 @@ __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const 
         if (lane == 0) logits[e] = (bias && e < E) ? s + bias[e] : s;
     }
     __syncthreads();
-    if (warp == 0) {
-        if (gate && lane == 0) gate[n] = 1.f / (1.f + expf(-logits[E]));
-        if (softmax) {
-            float mx = -INFINITY;
-            for (int e = lane; e < E; e += 32) mx = fmaxf(mx, logits[e]);
-            mx = warp_max(mx);
-            float sum = 0.f;
-            for (int e = lane; e < E; e += 32) {
-                const float p = expf(logits[e] - mx);
-                score[e] = p;
-                sum += p;
-            }
-            sum = warp_sum(sum);
-            __syncwarp();
-            for (int e = lane; e < E; e += 32) {
-                const float p = score[e] / sum;
-                score[e] = p;
-                logits[e] = correction ? p + correction[e] : p;
-            }
-            __syncwarp();
-        } else if (correction) {
-            for (int e = lane; e < E; e += 32) {
-                score[e] = 1.f / (1.f + expf(-logits[e]));
-                logits[e] = score[e] + correction[e];
-            }
-            __syncwarp();
+    if (warp == 0) route_choose(logits, score, n, top, ids, wts, E, mode, correction, gate, lane);
+}
+
+// The same for steps of many rows: a block takes ROUTE_TOKENS tokens, so that the router matrix is read once for all of
+// them; a warp has four router outputs at a time and 32 sums (output, token), which are added over the lanes together.
+#define ROUTE_TOKENS 8
+__global__ void __launch_bounds__(256) route_topk_tile_kernel(const void* __restrict__ h, int h_bf16, const float* __restrict__ wr, int top,
+                                                              int* __restrict__ ids, float* __restrict__ wts, int N, int Hd, int E, int mode,
+                                                              const float* __restrict__ bias, const float* __restrict__ correction,
+                                                              float* __restrict__ gate) {
+    extern __shared__ float route_smem[];
+    pdl_wait();                                    // what the kernels before wrote is complete
+    pdl_trigger();
+    const int rows_w = gate ? E + 1 : E;
+    float* rows = route_smem;                                // [ROUTE_TOKENS][Hd]
+    float* logits = rows + ROUTE_TOKENS * Hd;                // [ROUTE_TOKENS][E + 1]
+    float* score = logits + ROUTE_TOKENS * (E + 1);          // [ROUTE_TOKENS][E]
+    const int n0 = blockIdx.x * ROUTE_TOKENS, cnt = min(ROUTE_TOKENS, N - n0);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int i = threadIdx.x; i < ROUTE_TOKENS * Hd; i += blockDim.x)
+        rows[i] = i < cnt * Hd ? load_as_float(h, h_bf16, (size_t)n0 * Hd + i) : 0.f;
+    __syncthreads();
+    for (int e0 = warp * 4; e0 < rows_w; e0 += 32) {
+        const float* w[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) w[k] = wr + (size_t)min(e0 + k, rows_w - 1) * Hd;
+        float acc[32];                                       // output k, token t at 8 k + t
+#pragma unroll
+        for (int i = 0; i < 32; ++i) acc[i] = 0.f;
+#pragma unroll 2
+        for (int i = lane; i < Hd; i += 32) {
+            float wv[4], x[8];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) wv[k] = w[k][i];
+#pragma unroll
+            for (int t = 0; t < 8; ++t) x[t] = rows[t * Hd + i];
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+#pragma unroll
+                for (int t = 0; t < 8; ++t) acc[8 * k + t] = fmaf(x[t], wv[k], acc[8 * k + t]);
         }
-        const bool by_score = softmax || correction;
-        float first = 0.f, total = 0.f;                      // mode 2: the largest logit, and the sum of the chosen exponentials
-        for (int k = 0; k < top; ++k) {
-            float best = -INFINITY;
-            int at = -1;
-            for (int e = lane; e < E; e += 32)
-                if (logits[e] > best) { best = logits[e]; at = e; }
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-                if (ob > best || (ob == best && oa >= 0 && (at < 0 || oa < at))) { best = ob; at = oa; }
+        // every exchange halves the values a lane holds: lane l ends with the sum of value l
+#pragma unroll
+        for (int m = 16; m > 0; m >>= 1) {
+            const bool up = lane & m;
+#pragma unroll
+            for (int i = 0; i < m; ++i) {
+                const float give = up ? acc[i] : acc[i + m], keep = up ? acc[i + m] : acc[i];
+                acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, m);
             }
-            if (lane == 0) {
-                ids[(size_t)n * top + k] = at;
-                float w;
-                if (mode == 2) {
-                    if (k == 0) first = best;
-                    w = expf(best - first);
-                    total += w;
-                } else {
-                    w = by_score ? score[at] : 1.f / (1.f + expf(-best));
-                }
-                wts[(size_t)n * top + k] = w;
-                logits[at] = -INFINITY;
-            }
-            __syncwarp();
         }
-        if (mode == 2) {
-            total = __shfl_sync(0xffffffffu, total, 0);
-            for (int k = lane; k < top; k += 32) wts[(size_t)n * top + k] /= total;
-        }
+        const int e = e0 + (lane >> 3);
+        if (e < rows_w) logits[(lane & 7) * (E + 1) + e] = (bias && e < E) ? acc[0] + bias[e] : acc[0];
     }
+    __syncthreads();
+    if (warp < cnt) route_choose(logits + warp * (E + 1), score + warp * E, n0 + warp, top, ids, wts, E, mode, correction, gate, lane);
 }
 
 // mode: 0 sigmoid scores, 1 softmax over the E router outputs, 2 softmax over the chosen logits. bias: float32 [E] or null. correction: float32 [E] or null. gate: float32 [N] or
@@ -120,22 +180,18 @@ LLMP_API int llmp_route_topk(const void* h, int h_dtype, const float* w_router, 
     LLMP_REQUIRE(E > 0 && top > 0 && top <= E && Hd > 0 && E <= 8192, "route_topk: bad sizes experts=%d top=%d width=%d", E, top, Hd);
     const size_t smem = (size_t)(2 * E + 1 + Hd) * sizeof(float);
     LLMP_REQUIRE(smem <= 200 * 1024, "route_topk: a row of %d entries does not fit shared memory", Hd);
+    const size_t tile_smem = (size_t)ROUTE_TOKENS * (2 * E + 1 + Hd) * sizeof(float);
+    if (N > 64 && tile_smem <= 200 * 1024) {
+        LLMP_ALLOW_SMEM(route_topk_tile_kernel, tile_smem);
+        llmp_launch_dependent(route_topk_tile_kernel, dim3((N + ROUTE_TOKENS - 1) / ROUTE_TOKENS), dim3(256), tile_smem, stream, h,
+                              (int)(h_dtype == LLMP_BF16), w_router, top, ids, wts, N, Hd, E, mode, bias, correction, gate);
+        return llmp_check_launch("route_topk");
+    }
     LLMP_ALLOW_SMEM(route_topk_kernel, smem);
     // few rows (a decode step): a warp per expert, so that the router matrix is read by many warps at once
     llmp_launch_dependent(route_topk_kernel, dim3(N), dim3(N <= 64 ? 1024 : 256), smem, stream, h, (int)(h_dtype == LLMP_BF16), w_router,
                           top, ids, wts, Hd, E, mode, bias, correction, gate);
     return llmp_check_launch("route_topk");
-}
-
-// form 0: clamped, the weight on the input; form 1: silu(g) u, the weight on the output; form 2: max(u, 0)^2 without a
-// gate, the weight on the output
-#define EXPERT_FORM_UNGATED 2
-__device__ __forceinline__ float expert_act(float g, float u, float w, float limit, int form) {
-    if (form == EXPERT_FORM_UNGATED) { u = fmaxf(u, 0.f); return w * (u * u); }
-    if (form == 1) return w * (g / (1.f + expf(-g))) * u;
-    g = fminf(w * g, limit);
-    u = fminf(fmaxf(w * u, -limit), limit);
-    return g * (1.f / (1.f + expf(-1.702f * g))) * (u + 1.f);
 }
 
 // Eight consecutive entries of a row as floats, by 16-byte loads (the rows are 16-byte aligned when their length is a

@@ -128,6 +128,10 @@ __device__ __forceinline__ void tma_load_page_box(void* smem_dst, const CUtensor
 // in the 128-byte swizzle; cached per matrix (gemm_stream.cu).
 int llmp_stream_tensor_map(const void* ptr, long rows, long k, long ld, int box_rows, int box_kb, CUtensorMap* out);
 
+// Tensor map over a [rows, K] bfloat16 row-major matrix with row pitch ld, read in boxes of box_rows x 64 elements in the
+// 128-byte swizzle; rows and columns out of range arrive as zeros; cached per matrix (gemm_tc.cu).
+int llmp_matrix_tensor_map(const void* ptr, long rows, long k, long ld, int box_rows, CUtensorMap* out);
+
 // Number of SMs of the current device (gemm_stream.cu).
 int llmp_sm_count();
 

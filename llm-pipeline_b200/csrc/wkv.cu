@@ -7,7 +7,7 @@
 // wkv_shift:  the mixes x_t + (x_(t-1) - x_t) mu_s of every token's row with the row before it, one matrix per s. The row
 //             before a step's first token lies in the request's slot.
 // wkv_decay:  the decays exp(-exp(W2 tanh(low) + w0)) from the float32 rows `low` of the first step of their projection.
-// wkv_scan:   the recurrence; a block per (request, head, 16 value columns).
+// wkv_scan:   the recurrence; a block per (request, head, 32 value columns), long prompts in segments side by side.
 // wkv_gate:   every head's o divided by its root mean square, times a weight per channel and silu of the gate.
 //
 // A request's state is one float32 vector [shift piece | scan piece], each piece two copies that take turns by the parity
@@ -117,7 +117,7 @@ __global__ void __launch_bounds__(128) wkv_decay_kernel(const float* __restrict_
 
 // ---- the recurrence --------------------------------------------------------------------------------------------------
 constexpr int WK_THREADS = 128;
-constexpr int WK_COLS = 16;       // value columns of a block: a warp has four, a half-warp two
+constexpr int WK_COLS = 32;       // value columns of a block: a half-warp has four
 constexpr int WK_CHUNK = 8;       // tokens of a stage
 constexpr int WK_STAGES = 4;
 
@@ -125,10 +125,11 @@ struct WkvArgs {
     const float* r; const float* k; const float* v; long rkv_t;     // [tokens, H d] each, one stride
     const float* w; long w_t;                                        // [tokens, H d]
     const float* u;                                                  // [H, d]
-    float* state; long state_slot; long state_half;                  // a copy: [H][column blocks][2 NR][128] (see below)
+    float* state; long state_slot; long state_half;                  // a copy: [H][column blocks][4 NR][128] (see below)
     const int* q_start; const int* slots; const int* positions;
     float* o; long o_t;                                              // [tokens, H d]
-    int H, d, vec;
+    float* ends; float* decays; int seg_tokens, segments;            // segments: [requests][segments][a copy], [requests][segments][H][16 NR]
+    int H, d, vec, blocks;                                           // blocks: column blocks of a head
 };
 
 __device__ __forceinline__ void wk_cp4(float* dst, const float* src) {
@@ -154,58 +155,99 @@ template <int NR> __device__ __forceinline__ void wk_rows(const float* p, float 
     }
 }
 
-// A block owns (request, head, 16 value columns) and walks the request's tokens in order. A half-warp owns two columns; its
-// lane l holds their rows l NR .. l NR + NR - 1 in registers (16 NR >= d; rows past d stay zero because their keys are).
-// Nothing of a token's read-out feeds the recurrence, so the sums over the lanes of a chunk of 8 tokens are taken
-// together: 16 values (token, column) a lane, halved with every exchange, until each lane holds the value it stores.
+// A block owns (request, head, 32 value columns) and walks the request's tokens in order. A half-warp owns four columns;
+// its lane l holds their rows l NR .. l NR + NR - 1 in registers (16 NR >= d; rows past d stay zero because their keys
+// are). Nothing of a token's read-out feeds the recurrence, so the sums over the lanes of a chunk of 8 tokens are taken
+// together: 32 values (token, column) a lane, halved with every exchange, until each lane holds the two it stores.
 // The tokens' inputs come through a ring of stages of one chunk (asynchronous copies, one barrier a chunk).
-// In the slot a copy of the state is kept in the order in which the threads hold it: entry e = 2 i + column (i the row
-// within the lane) of thread t of column block b of head h at ((h blocks + b) 2 NR + e) 128 + t.
-template <int NR>
+// A copy of the state is kept in the order in which the threads hold it: entry e = 4 i + column (i the row within the lane)
+// of thread t of column block b of head h at ((h blocks + b) 4 NR + e) 128 + t.
+//
+// The recurrence is linear in its state, so a long prompt can be cut into segments of `seg_tokens` that run side by side
+// (blockIdx.z also counts segments). MODE 0: a segment after the first starts from zero, and every segment leaves its end
+// state and the products of its decays. MODE 1, for the segments after the first: the state a segment really starts
+// from, folded from the earlier segments' ends, adds (the decays since the segment's start, times r)^T state to the
+// segment's read-outs; the last segment's block writes the request's state.
+template <int NR, int MODE>
 __global__ void __launch_bounds__(WK_THREADS) wkv_scan_kernel(const WkvArgs a) {
     constexpr int DP = 16 * NR;                          // rows with padding
     constexpr int ROW = 3 * DP + WK_COLS;                // r, k, w, this block's v
+    constexpr int E = 4 * NR;                            // state entries of a thread
     extern __shared__ __align__(16) float wk_smem[];
     float* us = wk_smem;                                 // [DP]
     float* ring = us + DP;                               // [WK_STAGES][WK_CHUNK][ROW]
     pdl_wait();
     pdl_trigger();
-    const int q = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
-    const int begin = a.q_start[q], end = a.q_start[q + 1];
+    const int q = blockIdx.x, h = blockIdx.y, b = blockIdx.z % a.blocks;
+    const int seg = blockIdx.z / a.blocks + (MODE == 1 ? 1 : 0);
+    const int req_begin = a.q_start[q], req_end = a.q_start[q + 1];
+    const int begin = req_begin + seg * a.seg_tokens;    // without segments seg is 0 and seg_tokens covers every request
+    const int end = min(req_end, begin + a.seg_tokens);
     if (end <= begin) return;
     const int tid = threadIdx.x, lane = tid & 31, l16 = lane & 15;
     const int d = a.d, j0 = b * WK_COLS;
     const int ncols = min(WK_COLS, d - j0);
-    const int col = (tid >> 4) * 2;                      // this thread's first column within the block
-    const int p0 = a.positions[begin];
-    float* slot = a.state + (size_t)a.slots[q] * a.state_slot + ((size_t)h * gridDim.z + b) * (2 * NR) * WK_THREADS + tid;
-    const float* rd = slot + ((p0 + 1) & 1) * a.state_half;
-    float* wr = slot + ((p0 + end - begin - 1) & 1) * a.state_half;
-    float S[NR][2];
+    const int col = (tid >> 4) * 4;                      // this thread's first column within the block
+    const int p0 = a.positions[req_begin];
+    const size_t place = ((size_t)h * a.blocks + b) * E * WK_THREADS + tid;
+    const size_t copy = (size_t)a.H * a.blocks * E * WK_THREADS;
+    float* slot = a.state + (size_t)a.slots[q] * a.state_slot + place;
+    float* wr = slot + ((p0 + req_end - req_begin - 1) & 1) * a.state_half;
+    float* ends = a.ends + (size_t)q * a.segments * copy + place;                        // segment s at ends + s * copy
+    float* decays = a.decays + ((size_t)q * a.segments * a.H + h) * DP + l16 * NR;       // segment s at decays + s * H * DP
+    float S[NR][4], p[NR];                               // p: products of the decays since the segment's start
 #pragma unroll
-    for (int i = 0; i < NR; ++i) {
-        S[i][0] = rd[(size_t)(2 * i) * WK_THREADS];
-        S[i][1] = rd[(size_t)(2 * i + 1) * WK_THREADS];
+    for (int i = 0; i < NR; ++i) p[i] = 1.f;
+    if (MODE == 1) {
+        // the state this segment starts from: the first segment's end, then the later ones before this one
+#pragma unroll
+        for (int e = 0; e < E; ++e) S[e >> 2][e & 3] = ends[(size_t)e * WK_THREADS];
+        for (int s = 1; s < seg; ++s) {
+            float f[NR];
+            wk_rows<NR>(decays + (size_t)s * a.H * DP, f);
+#pragma unroll
+            for (int e = 0; e < E; ++e) S[e >> 2][e & 3] = fmaf(f[e >> 2], S[e >> 2][e & 3], ends[s * copy + (size_t)e * WK_THREADS]);
+        }
+        if (end == req_end) {
+            float f[NR];
+            wk_rows<NR>(decays + (size_t)seg * a.H * DP, f);
+#pragma unroll
+            for (int e = 0; e < E; ++e)
+                wr[(size_t)e * WK_THREADS] = fmaf(f[e >> 2], S[e >> 2][e & 3], ends[seg * copy + (size_t)e * WK_THREADS]);
+        }
+    } else if (seg == 0) {
+        const float* rd = slot + ((p0 + 1) & 1) * a.state_half;
+#pragma unroll
+        for (int e = 0; e < E; ++e) S[e >> 2][e & 3] = rd[(size_t)e * WK_THREADS];
+    } else {
+#pragma unroll
+        for (int e = 0; e < E; ++e) S[e >> 2][e & 3] = 0.f;
     }
     for (int i = tid; i < DP; i += WK_THREADS) us[i] = i < d ? a.u[(size_t)h * d + i] : 0.f;
     if (d < DP || ncols < WK_COLS)
         for (int i = tid; i < WK_STAGES * WK_CHUNK * ROW; i += WK_THREADS) ring[i] = 0.f;       // the padding stays as it is now
     __syncthreads();
     const int chunks = (end - begin + WK_CHUNK - 1) / WK_CHUNK;
+    // a lane's pieces of a token (16 bytes where all rows allow it) are the same for all tokens; a warp takes every fourth token
+    const int unit = a.vec ? 4 : 1, du = d / unit, per = 3 * du + (MODE == 1 ? 0 : ncols / unit);
     auto issue = [&](int s) {
         if (s < chunks) {
             float* base = ring + (size_t)(s % WK_STAGES) * WK_CHUNK * ROW;
             const int t0 = begin + s * WK_CHUNK, cnt = min(WK_CHUNK, end - t0);
-            const int unit = a.vec ? 4 : 1, du = d / unit, per = 3 * du + ncols / unit;      // pieces of a row of r, k, w; of a token
-            for (int x = lane; x < per; x += 32) {       // a lane's pieces are the same for all tokens; a warp takes every fourth token
+            for (int x = lane; x < per; x += 32) {
                 const int which = (x >= du) + (x >= 2 * du) + (x >= 3 * du);
+                if (MODE == 1 && which == 1) continue;   // the correction reads no keys
                 const int at = (x - which * du) * unit;
                 const float* src = (which == 0 ? a.r : which == 1 ? a.k : which == 2 ? a.w : a.v + j0) + (size_t)h * d + at;
                 const long stride = which == 2 ? a.w_t : a.rkv_t;
-                for (int tt = tid >> 5; tt < cnt; tt += WK_THREADS / 32) {
-                    float* dst = base + (size_t)tt * ROW + which * DP + at;
-                    if (a.vec) wk_cp16(dst, src + (size_t)(t0 + tt) * stride);
-                    else wk_cp4(dst, src + (size_t)(t0 + tt) * stride);
+                float* dst = base + which * DP + at;
+#pragma unroll
+                for (int tt0 = 0; tt0 < WK_CHUNK; tt0 += WK_THREADS / 32) {
+                    const int tt = tt0 + (tid >> 5);
+                    if (tt < cnt) {
+                        if (a.vec) wk_cp16(dst + (size_t)tt * ROW, src + (size_t)(t0 + tt) * stride);
+                        else wk_cp4(dst + (size_t)tt * ROW, src + (size_t)(t0 + tt) * stride);
+                    }
                 }
             }
         }
@@ -215,66 +257,116 @@ __global__ void __launch_bounds__(WK_THREADS) wkv_scan_kernel(const WkvArgs a) {
     wk_rows<NR>(us + l16 * NR, ul);
 #pragma unroll
     for (int s = 0; s < WK_STAGES - 1; ++s) issue(s);
+    struct Inputs { float r[NR], k[NR], w[NR]; float4 v; };
+    auto fetch = [&](const float* cur, Inputs& x) {
+        wk_rows<NR>(cur + l16 * NR, x.r);
+        wk_rows<NR>(cur + 2 * DP + l16 * NR, x.w);
+        if (MODE == 0) {
+            wk_rows<NR>(cur + DP + l16 * NR, x.k);
+            x.v = *reinterpret_cast<const float4*>(cur + 3 * DP + col);
+        }
+    };
+    auto token = [&](const Inputs& x, float (&o)[4]) {
+        if (MODE == 1) {
+            o[0] = o[1] = o[2] = o[3] = 0.f;
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const float rp = x.r[i] * p[i];
+                p[i] *= x.w[i];
+#pragma unroll
+                for (int c = 0; c < 4; ++c) o[c] = fmaf(rp, S[i][c], o[c]);
+            }
+            return;
+        }
+        const float v[4] = {x.v.x, x.v.y, x.v.z, x.v.w};
+        float ruk = 0.f;
+#pragma unroll
+        for (int i = 0; i < NR; ++i) ruk = fmaf(x.r[i], ul[i] * x.k[i], ruk);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) o[c] = ruk * v[c];
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                o[c] = fmaf(x.r[i], S[i][c], o[c]);
+                S[i][c] = fmaf(x.w[i], S[i][c], x.k[i] * v[c]);
+            }
+            p[i] *= x.w[i];
+        }
+    };
+    float* out = a.o + (size_t)h * d + j0;
     for (int s = 0; s < chunks; ++s) {
         asm volatile("cp.async.wait_group %0;\n" ::"n"(WK_STAGES - 2) : "memory");
         __syncthreads();                                 // stage s is here for everyone; everyone has left stage s - 1
-        issue(s + WK_STAGES - 1);                        // into the buffer of stage s - 1
         const float* base = ring + (size_t)(s % WK_STAGES) * WK_CHUNK * ROW;
         const int t0 = begin + s * WK_CHUNK, cnt = min(WK_CHUNK, end - t0);
-        auto token = [&](const float* cur, float& o0, float& o1) {
-            float r[NR], k[NR], w[NR];
-            wk_rows<NR>(cur + l16 * NR, r);
-            wk_rows<NR>(cur + DP + l16 * NR, k);
-            wk_rows<NR>(cur + 2 * DP + l16 * NR, w);
-            const float2 v = *reinterpret_cast<const float2*>(cur + 3 * DP + col);
-            float ruk = 0.f;
-            o0 = o1 = 0.f;
-#pragma unroll
-            for (int i = 0; i < NR; ++i) {
-                ruk = fmaf(r[i], ul[i] * k[i], ruk);
-                o0 = fmaf(r[i], S[i][0], o0);
-                o1 = fmaf(r[i], S[i][1], o1);
-                S[i][0] = fmaf(w[i], S[i][0], k[i] * v.x);
-                S[i][1] = fmaf(w[i], S[i][1], k[i] * v.y);
-            }
-            o0 = fmaf(ruk, v.x, o0);
-            o1 = fmaf(ruk, v.y, o1);
-        };
         if (cnt == WK_CHUNK) {
-            float acc[2 * WK_CHUNK];                     // (token tt, column c) at 2 tt + c
+            float acc[4 * WK_CHUNK];                     // (token tt, column c) at 4 tt + c
+            Inputs x[2];
+            fetch(base, x[0]);
+            issue(s + WK_STAGES - 1);                    // into the buffer of stage s - 1
+            // lane l16 ends with values 2 l16 and 2 l16 + 1: token l16 / 2, columns 2 (l16 & 1) and the next
+            const int jo = col + 2 * (l16 & 1);
+            float* dst = out + (size_t)(t0 + (l16 >> 1)) * a.o_t + jo;
+            float old0 = 0.f, old1 = 0.f;
+            if (MODE == 1) {
+                if (jo < ncols) old0 = dst[0];
+                if (jo + 1 < ncols) old1 = dst[1];
+            }
 #pragma unroll
-            for (int tt = 0; tt < WK_CHUNK; ++tt) token(base + (size_t)tt * ROW, acc[2 * tt], acc[2 * tt + 1]);
-            // lane l16 ends with the sum of value l16: bit m of the lane chooses the half that keeps going
+            for (int tt = 0; tt < WK_CHUNK; ++tt) {
+                if (tt + 1 < WK_CHUNK) fetch(base + (size_t)(tt + 1) * ROW, x[(tt + 1) & 1]);      // a token ahead of the sums
+                float o[4];
+                token(x[tt & 1], o);
 #pragma unroll
-            for (int m = 8; m > 0; m >>= 1) {
-                const bool up = l16 & m;
+                for (int c = 0; c < 4; ++c) acc[4 * tt + c] = o[c];
+            }
+            // bit m / 2 of the lane chooses the half that keeps going
+#pragma unroll
+            for (int m = 16; m > 1; m >>= 1) {
+                const bool up = l16 & (m >> 1);
 #pragma unroll
                 for (int i = 0; i < m; ++i) {
                     const float give = up ? acc[i] : acc[i + m], keep = up ? acc[i + m] : acc[i];
-                    acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, m);
+                    acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, m >> 1);
                 }
             }
-            const int j = col + (l16 & 1);
-            if (j < ncols) a.o[(size_t)(t0 + (l16 >> 1)) * a.o_t + (size_t)h * d + j0 + j] = acc[0];
+            if (jo < ncols) dst[0] = acc[0] + old0;
+            if (jo + 1 < ncols) dst[1] = acc[1] + old1;
         } else {
+            issue(s + WK_STAGES - 1);
             for (int tt = 0; tt < cnt; ++tt) {
-                float o0, o1;
-                token(base + (size_t)tt * ROW, o0, o1);
+                Inputs x;
+                fetch(base + (size_t)tt * ROW, x);
+                float o[4];
+                token(x, o);
 #pragma unroll
                 for (int m = 8; m > 0; m >>= 1) {
-                    o0 += __shfl_xor_sync(0xffffffffu, o0, m);
-                    o1 += __shfl_xor_sync(0xffffffffu, o1, m);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) o[c] += __shfl_xor_sync(0xffffffffu, o[c], m);
                 }
-                if (l16 < 2 && col + l16 < ncols) a.o[(size_t)(t0 + tt) * a.o_t + (size_t)h * d + j0 + col + l16] = l16 ? o1 : o0;
+                if (l16 < 4 && col + l16 < ncols) {
+                    float* dst = out + (size_t)(t0 + tt) * a.o_t + col + l16;
+                    const float sum = l16 == 0 ? o[0] : l16 == 1 ? o[1] : l16 == 2 ? o[2] : o[3];
+                    *dst = MODE == 1 ? *dst + sum : sum;
+                }
             }
         }
     }
     asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    if (MODE == 1) return;
+    if (seg > 0 || end < req_end) {                      // one of several segments
+        float* to = ends + seg * copy;
 #pragma unroll
-    for (int i = 0; i < NR; ++i) {
-        wr[(size_t)(2 * i) * WK_THREADS] = S[i][0];
-        wr[(size_t)(2 * i + 1) * WK_THREADS] = S[i][1];
+        for (int e = 0; e < E; ++e) to[(size_t)e * WK_THREADS] = S[e >> 2][e & 3];
+        if (b == 0 && tid < 16) {
+#pragma unroll
+            for (int i = 0; i < NR; ++i) decays[(size_t)seg * a.H * DP + i] = p[i];
+        }
+        return;
     }
+#pragma unroll
+    for (int e = 0; e < E; ++e) wr[(size_t)e * WK_THREADS] = S[e >> 2][e & 3];
 }
 
 int wkv_rows_per_lane(int d) {
@@ -361,12 +453,19 @@ LLMP_API int llmp_wkv_decay(const float* low, long low_t, const float* w2t, cons
 // Entries of one copy of the recurrence's state (0: heads of this size are not served).
 LLMP_API long llmp_wkv_state_entries(int H, int d) {
     if (H <= 0 || d <= 0 || d > 256) return 0;
-    return (long)H * ((d + WK_COLS - 1) / WK_COLS) * 2 * wkv_rows_per_lane(d) * WK_THREADS;
+    return (long)H * ((d + WK_COLS - 1) / WK_COLS) * 4 * wkv_rows_per_lane(d) * WK_THREADS;
 }
 
+// Float32 scratch of a scan in `segments` segments per request.
+LLMP_API long llmp_wkv_scratch(int R, int H, int d, int segments) {
+    return (long)R * segments * (llmp_wkv_state_entries(H, d) + (long)H * 16 * wkv_rows_per_lane(d));
+}
+
+// segments > 1: requests are cut into that many segments of seg_tokens (they must cover the longest), with `scratch` of
+// llmp_wkv_scratch floats.
 LLMP_API int llmp_wkv_scan(const float* r, const float* k, const float* v, long rkv_t, const float* w, long w_t, const float* u, float* state,
                            long state_slot, long state_half, const int* q_start, const int* slots, const int* positions, float* o,
-                           long o_t, int R, int H, int d, cudaStream_t stream) {
+                           long o_t, int R, int H, int d, int segments, int seg_tokens, float* scratch, cudaStream_t stream) {
     if (R <= 0) return 0;
     LLMP_REQUIRE(H > 0 && H <= 65535 && d > 0 && d <= 256, "wkv_scan: %d heads of %d channels are not served", H, d);
     LLMP_REQUIRE(state_half >= llmp_wkv_state_entries(H, d), "wkv_scan: the state's copies are too small");
@@ -375,12 +474,24 @@ LLMP_API int llmp_wkv_scan(const float* r, const float* k, const float* v, long 
     a.state_half = state_half; a.q_start = q_start; a.slots = slots; a.positions = positions; a.o = o; a.o_t = o_t; a.H = H; a.d = d;
     a.vec = d % 4 == 0 && rkv_t % 4 == 0 && w_t % 4 == 0 && ((size_t)r | (size_t)k | (size_t)v | (size_t)w) % 16 == 0;
     const int nr = wkv_rows_per_lane(d);
+    a.blocks = (d + WK_COLS - 1) / WK_COLS;
+    const bool cut = segments > 1;
+    LLMP_REQUIRE(!cut || (scratch && (size_t)scratch % 16 == 0 && seg_tokens > 0 && seg_tokens % WK_CHUNK == 0 && (long)segments * a.blocks <= 65535),
+                 "wkv_scan: segments need scratch and a length that is a multiple of %d", WK_CHUNK);
+    a.segments = cut ? segments : 1;
+    a.seg_tokens = cut ? seg_tokens : 0x3fffffff;
+    a.ends = scratch;
+    a.decays = cut ? scratch + (size_t)R * segments * llmp_wkv_state_entries(H, d) : nullptr;
     const size_t smem = sizeof(float) * ((size_t)16 * nr + (size_t)WK_STAGES * WK_CHUNK * (48 * nr + WK_COLS));
-    const dim3 grid(R, H, (d + WK_COLS - 1) / WK_COLS);
-#define LLMP_WKV(NR)                                                                             \
-    if (nr == NR) {                                                                              \
-        LLMP_ALLOW_SMEM(wkv_scan_kernel<NR>, smem);                                              \
-        llmp_launch_dependent(wkv_scan_kernel<NR>, grid, dim3(WK_THREADS), smem, stream, a);     \
+    const dim3 grid(R, H, a.blocks * a.segments), later(R, H, a.blocks * (a.segments - 1));
+#define LLMP_WKV(NR)                                                                                        \
+    if (nr == NR) {                                                                                         \
+        LLMP_ALLOW_SMEM((wkv_scan_kernel<NR, 0>), smem);                                                    \
+        llmp_launch_dependent(wkv_scan_kernel<NR, 0>, grid, dim3(WK_THREADS), smem, stream, a);             \
+        if (cut) {                                                                                          \
+            LLMP_ALLOW_SMEM((wkv_scan_kernel<NR, 1>), smem);                                                \
+            llmp_launch_dependent(wkv_scan_kernel<NR, 1>, later, dim3(WK_THREADS), smem, stream, a);        \
+        }                                                                                                   \
     } else
     LLMP_WKV(1) LLMP_WKV(2) LLMP_WKV(4) LLMP_WKV(8) LLMP_WKV(16) {}
 #undef LLMP_WKV

@@ -81,6 +81,7 @@ _SIGNATURES = {
     "llmp_convert_rows": [_P, _L, _P, _I, _L, _I, _P],
     "llmp_route_topk": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P, _P],
     "llmp_expert_grouped": [_P, _P, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "llmp_expert_tc": [_P, _P, _P, _P, _P, _F, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "llmp_expert_rows": [_P, _P, _P, _I, _P, _P, _F, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "llmp_add_layernorm": [_P, _P, _I, _P, _I, _P, _P, _I, _F, _P, _I, _I, _I, _P, _P],
     "llmp_relu_squared": [_P, _P, _I, _L, _P],
@@ -99,7 +100,7 @@ _SIGNATURES = {
     "llmp_sigmoid_attention_mma": [_P, _L, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _P, _L, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "llmp_wkv_shift": [_P, _P, _P, _L, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
     "llmp_wkv_decay": [_P, _L, _P, _P, _P, _I, _I, _I, _P],
-    "llmp_wkv_scan": [_P, _P, _P, _L, _P, _L, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _P],
+    "llmp_wkv_scan": [_P, _P, _P, _L, _P, _L, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _P],
     "llmp_wkv_gate": [_P, _L, _P, _L, _P, _P, _I, _L, _I, _I, _I, _F, _P],
     "llmp_xielu": [_P, _P, _I, _F, _F, _P, _I, _L, _I, _P],
     "llmp_scaled_sum": [_P, _F, _P, _F, _P, _L, _P],
@@ -995,6 +996,7 @@ def expert_rows(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     return out
 
 
+EXPERT_TC_MIN_ROWS = 512             # pairs from which those products are the tcgen05 ones
 EXPERT_GROUPED_MIN_ROWS = 33         # (token, choice) pairs from which a step's experts run as grouped products
 
 
@@ -1030,11 +1032,48 @@ def expert_grouped(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tenso
     return out
 
 
+def expert_tc_supports(dtype: torch.dtype, Hd: int, F: int) -> bool:
+    if dtype != torch.bfloat16:
+        return False
+    fn = library().llmp_expert_tc_supports
+    fn.argtypes = [_I, _I]
+    fn.restype = _I
+    return bool(fn(Hd, F))
+
+
+def expert_tc(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
+              limit: float, out: torch.Tensor, form: str = "clamped", identity: int = 0) -> torch.Tensor:
+    """``expert_grouped`` with tcgen05 products (csrc/routed_experts_tc.cu): tiles of 128 pairs of one expert, the tokens' rows
+    gathered into the sorted order first."""
+    N, Hd = h.shape
+    E, rows_f, _ = w_gate_up.shape
+    F = rows_f if form in UNGATED_EXPERT_FORMS else rows_f // 2
+    top = ids.shape[1]
+    _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and rows_f == (F if form in UNGATED_EXPERT_FORMS else 2 * F) and
+          w_gate_up.shape[2] == Hd and w_down.shape == (E, Hd, F) and h.dtype == w_gate_up.dtype == w_down.dtype == torch.bfloat16,
+          "expert matrices have the wrong layout")
+    _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape == (N, Hd), "expert output must be float32 [tokens, width]")
+    fn = library().llmp_expert_tc_rows
+    fn.argtypes = [_I, _I]
+    fn.restype = _L
+    rows = int(fn(N * top, E))
+    ints = torch.empty(1 + rows // 128 + rows, dtype=torch.int32, device=h.device)
+    x = torch.empty((rows, Hd), dtype=torch.bfloat16, device=h.device)
+    y = torch.empty((rows, F), dtype=torch.bfloat16, device=h.device)
+    pair_out = torch.empty((N * top, Hd), dtype=torch.float32, device=h.device)
+    _call("llmp_expert_tc", _ptr(h), _ptr(w_gate_up), _ptr(w_down), _ptr(ids), _ptr(weights), float(limit), _ptr(ints), _ptr(x), _ptr(y),
+          _ptr(pair_out), _ptr(out), N, top, Hd, F, E, EXPERT_FORMS[form], int(identity), error_flag().data_ptr(), _stream())
+    return out
+
+
 def routed_experts(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
                    limit: float, out: torch.Tensor, form: str = "clamped", identity: int = 0) -> torch.Tensor:
     """The experts' work for a step's rows, by the kernel that suits their number: grouped tensor-core products for many
-    bfloat16 rows, a warp per output entry (``expert_rows``) for the few rows of a decode step and for float32."""
+    bfloat16 rows (tcgen05 from ``EXPERT_TC_MIN_ROWS`` pairs on), a warp per output entry (``expert_rows``) for the few rows of
+    a decode step and for float32."""
     pairs = ids.numel()
+    if pairs >= EXPERT_TC_MIN_ROWS and expert_tc_supports(h.dtype, h.shape[1], w_down.shape[2]):
+        return expert_tc(h, w_gate_up, w_down, ids, weights, limit, out, form, identity)
     if pairs >= EXPERT_GROUPED_MIN_ROWS and expert_grouped_supports(h.dtype, h.shape[1], w_down.shape[2]):
         return expert_grouped(h, w_gate_up, w_down, ids, weights, limit, out, form, identity)
     return expert_rows(h, w_gate_up, w_down, ids, weights, limit, out, form)
@@ -1713,12 +1752,26 @@ WKV_MAX_DIM = 256
 
 
 def wkv_state_entries(heads: int, dim: int) -> int:
-    """Entries of one copy of the wkv recurrence's state as csrc/wkv.cu keeps it: per head and block of 16 value columns, two
+    """Entries of one copy of the wkv recurrence's state as csrc/wkv.cu keeps it: per head and block of 32 value columns, four
     columns of ``rows`` rows for each of 16 lanes of 8 half-warps (16 ``rows`` >= dim, a power of two)."""
+    return heads * -(-dim // 32) * 4 * _wkv_rows(dim) * 128
+
+
+def _wkv_rows(dim: int) -> int:
     rows = 1
     while 16 * rows < dim:
         rows *= 2
-    return heads * -(-dim // 16) * 2 * rows * 128
+    return rows
+
+
+WKV_SEGMENT_TOKENS = 256             # tokens of a segment of a prompt whose segments run side by side
+
+
+def wkv_segments(longest: int, requests: int, heads: int, dim: int) -> int:
+    """Into how many segments a step cuts its requests: long portions whose blocks alone would leave most of the GPU's warps idle."""
+    if longest < 2 * WKV_SEGMENT_TOKENS or requests * heads * -(-dim // 32) >= 6 * sm_count():
+        return 1
+    return -(-longest // WKV_SEGMENT_TOKENS)
 
 
 def wkv_shift(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, state_offset: int, q_start: torch.Tensor, slots: torch.Tensor,
@@ -1752,9 +1805,11 @@ def wkv_decay(low: torch.Tensor, w2t: torch.Tensor, w0: torch.Tensor, out: torch
 
 def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, bonus: torch.Tensor, state: torch.Tensor,
              state_offset: int, q_start: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor, out: torch.Tensor, heads: int,
-             dim: int) -> torch.Tensor:
+             dim: int, segments: int = 1) -> torch.Tensor:
     """The wkv recurrence over the step's tokens, request by request (csrc/wkv.cu): ``r``, ``k``, ``v``, ``decay``, ``out`` float32
-    [tokens, heads dim], ``bonus`` float32 [heads, dim]. The state piece holds two copies of ``wkv_state_entries`` floats."""
+    [tokens, heads dim], ``bonus`` float32 [heads, dim]. The state piece holds two copies of ``wkv_state_entries`` floats.
+    ``segments`` > 1: every request is cut into that many segments of ``WKV_SEGMENT_TOKENS`` tokens that run side by side
+    (they must cover the longest), and a second launch adds what the earlier segments' states give."""
     N = r.shape[0]
     for t, name in ((r, "r"), (k, "k"), (v, "v"), (decay, "decay"), (out, "out")):
         _need(t.dtype == torch.float32 and t.stride(1) == 1 and t.shape == (N, heads * dim), f"wkv_scan: {name} must be float32 [tokens, heads dim]")
@@ -1762,9 +1817,14 @@ def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Ten
     _need(bonus.dtype == torch.float32 and bonus.is_contiguous() and bonus.shape == (heads, dim), "wkv_scan: the bonus must be float32 [heads, dim]")
     for t, name in ((q_start, "q_start"), (slots, "slots"), (positions, "positions")):
         _i32(t, name)
-    ptr, slot_stride, half = _state_views(state, state_offset, wkv_state_entries(heads, dim), "wkv_scan")
+    entries = wkv_state_entries(heads, dim)
+    ptr, slot_stride, half = _state_views(state, state_offset, entries, "wkv_scan")
+    scratch = None
+    if segments > 1:
+        scratch = torch.empty(slots.numel() * segments * (entries + heads * 16 * _wkv_rows(dim)), dtype=torch.float32, device=r.device)
     _call("llmp_wkv_scan", _ptr(r), _ptr(k), _ptr(v), r.stride(0), _ptr(decay), decay.stride(0), _ptr(bonus), ptr, slot_stride, half,
-          _ptr(q_start), _ptr(slots), _ptr(positions), _ptr(out), out.stride(0), slots.numel(), heads, dim, _stream())
+          _ptr(q_start), _ptr(slots), _ptr(positions), _ptr(out), out.stride(0), slots.numel(), heads, dim, int(segments), WKV_SEGMENT_TOKENS,
+          _ptr(scratch), _stream())
     return out
 
 

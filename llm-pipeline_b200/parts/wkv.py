@@ -92,7 +92,7 @@ class WKV(Mixer):
         decay = kernels.wkv_decay(low, self.w2t, self.w0, torch.empty((N, C), dtype=torch.float32, device=x.device))
         o = torch.empty((N, C), dtype=torch.float32, device=x.device)
         kernels.wkv_scan(r, k, v, decay, self.bonus, cache.state, 2 * self.hidden_size, ctx.q_start, ctx.slots, ctx.positions, o,
-                         self.heads, self.dim)
+                         self.heads, self.dim, kernels.wkv_segments(ctx.max_q_len, ctx.num_requests, self.heads, self.dim))
         gated = torch.empty((N, C), dtype=ctx.dtype, device=x.device)
         kernels.wkv_gate(o, z, self.norm_w, gated, self.heads, self.dim, self.eps)
         return linear(gated, self.w_out, out_dtype=torch.float32), None
