@@ -200,7 +200,9 @@ class ZasudraConfig(ModelConfig):
                 mixer = PartSpec("wkv", {"hidden_size": D, "heads": int(m["heads"]), "dim": int(m["dim"]), "eps": self.norm_eps}, f"{p}.mix")
             else:
                 mixer = self._attention(m, f"{p}.mix", positions, layer["type"] == "attention")
-            norms = {"mixer_out": PartSpec("rms_norm", {"size": D, "eps": self.norm_eps, "name": f"{p}.norm1", "gain": self.residual_mult})}
+            spare = [] if mlp is not None else [f"{p}.norm2"]           # a checkpoint may hold it for a layer without a feed-forward
+            norms = {"mixer_out": PartSpec("rms_norm", {"size": D, "eps": self.norm_eps, "name": f"{p}.norm1", "gain": self.residual_mult,
+                                                        "unused": spare})}
             feed_forward = None
             if mlp is not None:
                 feed_forward = PartSpec("routed_experts", {

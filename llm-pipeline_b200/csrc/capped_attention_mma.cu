@@ -7,7 +7,7 @@
 // the group. A cached row is [key | value]. Each of the four warps owns 16 rows and keeps their running softmax and output
 // in registers. Keys are walked in tiles of 64 aligned to key 0 (the same operations for a row however the prompt was
 // cut): first the tiles of the kept first tokens that lie before the window of the tile's first token, then from that
-// window's first key to the last token's own; half tiles that no row of a warp sees are skipped, rows of pages that
+// window's first key to the last token's own; tiles that no row of a warp sees are skipped, rows of pages that
 // are gone are never read. Per score: scale, cap (tanh by the special-function unit), the head's slope times the
 // distance, the mask; the softmax runs in units of log2 and starts from the sink (a key of that score without a value).
 // The gate, sigmoid of a float32 row, is applied as the output is stored.
@@ -249,6 +249,7 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
         }
         buf_issue = buf_issue + 1 == stages ? 0 : buf_issue + 1;
     }
+    unsigned qf[D16][4];                                         // this warp's query fragments, read once the copy is here
     int buf = 0;
     for (int j0 = first_tile; j0 <= hi; j0 = next_tile(j0)) {
         if (j_issue <= hi) {
@@ -266,6 +267,10 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
         else asm volatile("cp.async.wait_group 1;\n" ::: "memory");
         __syncthreads();
         const bf16* KVs = ring + (size_t)buf * STAGE_ELEMS;
+        if (j0 == first_tile) {
+#pragma unroll
+            for (int ks = 0; ks < D16; ++ks) cm_ldmatrix_x4(qf[ks], Qw + ks * 16);
+        }
         // the part of a tile that starts at its key `kbase` and has NB blocks of 8 keys: scores, softmax step, values
         auto part = [&](auto nbc, const int kbase) {
             constexpr int NB = decltype(nbc)::value;
@@ -280,15 +285,13 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
             for (int nb = 0; nb < NB; ++nb) s[nb][0] = s[nb][1] = s[nb][2] = s[nb][3] = 0.f;
 #pragma unroll
             for (int ks = 0; ks < D16; ++ks) {
-                unsigned qa[4];
-                cm_ldmatrix_x4(qa, Qw + ks * 16);
 #pragma unroll
                 for (int nb = 0; nb < NB; nb += 2) {
                     unsigned kf[4];
                     cm_ldmatrix_x4(kf, KVs + (size_t)(kbase + (nb + (lane >> 4)) * 8 + (lane & 7)) * KSTRIDE + ks * 16 +
                                            ((lane >> 3) & 1) * 8);
-                    cm_mma(s[nb], qa, kf[0], kf[1]);
-                    cm_mma(s[nb + 1], qa, kf[2], kf[3]);
+                    cm_mma(s[nb], qf[ks], kf[0], kf[1]);
+                    cm_mma(s[nb + 1], qf[ks], kf[2], kf[3]);
                 }
             }
             // scores in units of log2: scale (and cap), the distance bias, the mask
@@ -371,8 +374,7 @@ __global__ void __launch_bounds__(CM_THREADS, 2) capped_attention_mma_kernel(con
         if (split) {
             part(std::integral_constant<int, 2>{}, warp * 16);  // a quarter of the tile's keys for each of the four warps
         } else if (warp_has_rows) {
-            part(std::integral_constant<int, 4>{}, 0);
-            part(std::integral_constant<int, 4>{}, 32);
+            part(std::integral_constant<int, 8>{}, 0);
         }
         if (tid < CM_KEYS) key_off[buf][tid] = off_next;         // this round's tile was copied long ago: its places make room
         __syncthreads();                                         // the tile's buffer may be overwritten now

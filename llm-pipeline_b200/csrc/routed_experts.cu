@@ -19,6 +19,22 @@
 // reads an expert's rows once per 64 pairs (mma.sync); many rows go to routed_experts_tc.cu (tcgen05).
 #include "routed_experts.cuh"
 
+// Eight consecutive entries of a row as floats, by 16-byte loads (the rows are 16-byte aligned when their length is a
+// multiple of 8 and the tensors are).
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = __low2float(h2[i]);
+        v[2 * i + 1] = __high2float(h2[i]);
+    }
+}
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+
 // The choice of one token by one warp: `logits` [E (+ 1: the gate's)] in shared memory, overwritten; `score` [E] is scratch.
 __device__ __forceinline__ void route_choose(float* logits, float* score, int n, int top, int* __restrict__ ids, float* __restrict__ wts, int E,
                                              int mode, const float* __restrict__ correction, float* __restrict__ gate, int lane) {
@@ -89,9 +105,10 @@ __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const 
     pdl_wait();                                    // what the kernels before wrote is complete
     pdl_trigger();
     extern __shared__ float route_smem[];
-    float* logits = route_smem;                              // [E + 1]: logits, then what the choice goes by
-    float* score = route_smem + E + 1;                       // [E]: softmax scores (softmax only)
-    float* row = route_smem + 2 * E + 1;                     // [Hd]: the token's row, read once
+    float* row = route_smem;                                 // [Hd]: the token's row, read once
+    float* logits = row + Hd;                                // [E + 1]: logits, then what the choice goes by
+    float* score = logits + E + 1;                           // [E]: softmax scores (softmax only)
+    const bool vec = Hd % 8 == 0 && ((size_t)wr & 15) == 0;
     const int rows_w = gate ? E + 1 : E;                     // the gate's row follows the experts' rows
     const int n = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
@@ -99,11 +116,22 @@ __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const 
     __syncthreads();
     for (int e = warp; e < rows_w; e += nwarps) {
         const float* w = wr + (size_t)e * Hd;
-        // eight sums a lane, so that eight loads are in flight; their order of addition is fixed
+        // eight sums a lane, so that many loads are in flight; their order of addition is fixed
         float acc[8];
 #pragma unroll
         for (int u = 0; u < 8; ++u) acc[u] = 0.f;
         int i = lane;
+        if (vec) {
+#pragma unroll 4
+            for (int j = lane * 8; j < Hd; j += 256) {
+                float a[8], b[8];
+                load8(row + j, a);
+                load8(w + j, b);
+#pragma unroll
+                for (int u = 0; u < 8; ++u) acc[u] = fmaf(a[u], b[u], acc[u]);
+            }
+            i = Hd;
+        }
         for (; i + 7 * 32 < Hd; i += 256) {
 #pragma unroll
             for (int u = 0; u < 8; ++u) acc[u] = fmaf(row[i + 32 * u], w[i + 32 * u], acc[u]);
@@ -132,8 +160,20 @@ __global__ void __launch_bounds__(256) route_topk_tile_kernel(const void* __rest
     float* score = logits + ROUTE_TOKENS * (E + 1);          // [ROUTE_TOKENS][E]
     const int n0 = blockIdx.x * ROUTE_TOKENS, cnt = min(ROUTE_TOKENS, N - n0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int i = threadIdx.x; i < ROUTE_TOKENS * Hd; i += blockDim.x)
-        rows[i] = i < cnt * Hd ? load_as_float(h, h_bf16, (size_t)n0 * Hd + i) : 0.f;
+    const bool vec = Hd % 8 == 0 && (((size_t)h | (size_t)wr) & 15) == 0;
+    if (vec && h_bf16) {
+        const bf16* src = reinterpret_cast<const bf16*>(h) + (size_t)n0 * Hd;
+#pragma unroll 4
+        for (int i = threadIdx.x * 8; i < ROUTE_TOKENS * Hd; i += blockDim.x * 8) {
+            float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+            if (i < cnt * Hd) load8(src + i, v);
+            *reinterpret_cast<float4*>(rows + i) = make_float4(v[0], v[1], v[2], v[3]);
+            *reinterpret_cast<float4*>(rows + i + 4) = make_float4(v[4], v[5], v[6], v[7]);
+        }
+    } else {
+        for (int i = threadIdx.x; i < ROUTE_TOKENS * Hd; i += blockDim.x)
+            rows[i] = i < cnt * Hd ? load_as_float(h, h_bf16, (size_t)n0 * Hd + i) : 0.f;
+    }
     __syncthreads();
     for (int e0 = warp * 4; e0 < rows_w; e0 += 32) {
         const float* w[4];
@@ -142,17 +182,30 @@ __global__ void __launch_bounds__(256) route_topk_tile_kernel(const void* __rest
         float acc[32];                                       // output k, token t at 8 k + t
 #pragma unroll
         for (int i = 0; i < 32; ++i) acc[i] = 0.f;
+        int i0 = 0;
+        if (vec) {
 #pragma unroll 2
-        for (int i = lane; i < Hd; i += 32) {
-            float wv[4], x[8];
+            for (int i = lane * 4; i < Hd; i += 128) {       // four entries a lane and step
+                float4 wv[4];
 #pragma unroll
-            for (int k = 0; k < 4; ++k) wv[k] = w[k][i];
+                for (int k = 0; k < 4; ++k) wv[k] = *reinterpret_cast<const float4*>(w[k] + i);
 #pragma unroll
-            for (int t = 0; t < 8; ++t) x[t] = rows[t * Hd + i];
+                for (int t = 0; t < 8; ++t) {
+                    const float4 x = *reinterpret_cast<const float4*>(rows + t * Hd + i);
 #pragma unroll
-            for (int k = 0; k < 4; ++k)
+                    for (int k = 0; k < 4; ++k)
+                        acc[8 * k + t] = fmaf(x.w, wv[k].w, fmaf(x.z, wv[k].z, fmaf(x.y, wv[k].y, fmaf(x.x, wv[k].x, acc[8 * k + t]))));
+                }
+            }
+            i0 = Hd;
+        }
+        for (int i = i0 + lane; i < Hd; i += 32) {
 #pragma unroll
-                for (int t = 0; t < 8; ++t) acc[8 * k + t] = fmaf(x[t], wv[k], acc[8 * k + t]);
+            for (int k = 0; k < 4; ++k) {
+                const float wv = w[k][i];
+#pragma unroll
+                for (int t = 0; t < 8; ++t) acc[8 * k + t] = fmaf(rows[t * Hd + i], wv, acc[8 * k + t]);
+            }
         }
         // every exchange halves the values a lane holds: lane l ends with the sum of value l
 #pragma unroll
@@ -192,22 +245,6 @@ LLMP_API int llmp_route_topk(const void* h, int h_dtype, const float* w_router, 
     llmp_launch_dependent(route_topk_kernel, dim3(N), dim3(N <= 64 ? 1024 : 256), smem, stream, h, (int)(h_dtype == LLMP_BF16), w_router,
                           top, ids, wts, Hd, E, mode, bias, correction, gate);
     return llmp_check_launch("route_topk");
-}
-
-// Eight consecutive entries of a row as floats, by 16-byte loads (the rows are 16-byte aligned when their length is a
-// multiple of 8 and the tensors are).
-__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) {
-    const uint4 raw = *reinterpret_cast<const uint4*>(p);
-    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        v[2 * i] = __low2float(h2[i]);
-        v[2 * i + 1] = __high2float(h2[i]);
-    }
-}
-__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
-    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
 // grid (pairs, ceil(F / 8)): a warp per row of the expert's gate and up matrices (w_gu[e] = [gate rows; up rows], or the up

@@ -25,7 +25,7 @@ constexpr int MT_STAGES = 4;
 constexpr int MT_THREADS = 192;
 
 // One block. Shared: counts [E], cursor [E].
-__global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ ids, int pairs, int E, int* __restrict__ sorted_pair,
+__global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ ids, int pairs, int E, int rows, int* __restrict__ sorted_pair,
                                                         int* __restrict__ tile_expert, int* __restrict__ num_tiles) {
     extern __shared__ int ms_smem[];
     __shared__ int warp_sums[32], carry;
@@ -35,6 +35,7 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
     int* cursor = ms_smem + E;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     for (int e = tid; e < E; e += blockDim.x) counts[e] = 0;
+    for (int i = tid; i < rows; i += blockDim.x) sorted_pair[i] = -1;
     if (tid == 0) carry = 0;
     __syncthreads();
     for (int i = tid; i < pairs; i += blockDim.x) {
@@ -68,7 +69,6 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
         if (e < E) {
             cursor[e] = first * MT_ROWS;
             for (int k = 0; k < t; ++k) tile_expert[first + k] = e;
-            for (int i = first * MT_ROWS + n; i < (first + t) * MT_ROWS; ++i) sorted_pair[i] = -1;
         }
         __syncthreads();
         if (tid == 0) carry += warp_sums[31];
@@ -313,7 +313,8 @@ LLMP_API int llmp_expert_tc(const void* h, const void* w_first, const void* w_do
     int* sorted_pair = tile_expert + tiles_max;
     const size_t sort_smem = 2 * (size_t)E * sizeof(int);
     LLMP_ALLOW_SMEM(moe_sort_kernel, sort_smem);
-    llmp_launch_dependent(moe_sort_kernel, dim3(1), dim3(1024), sort_smem, stream, ids, pairs, E, sorted_pair, tile_expert, num_tiles);
+    llmp_launch_dependent(moe_sort_kernel, dim3(1), dim3(1024), sort_smem, stream, ids, pairs, E, (int)rows, sorted_pair,
+                          tile_expert, num_tiles);
     llmp_launch_dependent(moe_gather_kernel, dim3((unsigned)(rows / 4)), dim3(128), 0, stream, (const bf16*)h, (const int*)sorted_pair,
                           (const int*)num_tiles, top, Hd, (bf16*)x);
     MoeTcArgs a;

@@ -376,45 +376,40 @@ int wkv_rows_per_lane(int d) {
 }
 
 // ---- the heads' norm and the gate ------------------------------------------------------------------------------------
-// A warp per (token, head): out = o / sqrt(mean(o^2) + eps) * weight[channel] * silu(gate).
-__device__ __forceinline__ void store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
-__device__ __forceinline__ void store2(bf16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
-
-template <typename T>
+// out = o / sqrt(mean(o^2) + eps) * weight[channel] * silu(gate), the mean over the channels of a head. VEC: `group` lanes (a
+// power of two) share a head of at most 4 `group` channels, a lane has four of them; else a warp per (token, head).
+template <typename T, bool VEC>
 __global__ void wkv_gate_kernel(const float* __restrict__ o, long o_t, const float* __restrict__ gate, long gate_t,
-                                const float* __restrict__ weight, T* __restrict__ out, long out_t, long items, int H, int d, float eps) {
+                                const float* __restrict__ weight, T* __restrict__ out, long out_t, long items, int H, int d, int group, float eps) {
     pdl_wait();
     pdl_trigger();
-    const long item = (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (item >= items) return;
-    const int lane = threadIdx.x & 31;
-    const size_t t = (size_t)(item / H);
-    const int c0 = (int)(item % H) * d;
+    const long item = ((long)blockIdx.x * blockDim.x + threadIdx.x) / group;
+    const int lane = threadIdx.x % group;
+    const bool valid = item < items;
+    const size_t t = valid ? (size_t)(item / H) : 0;
+    const int c0 = valid ? (int)(item % H) * d : 0;
+    if (VEC) {
+        const int c = lane * 4;
+        const bool mine = valid && c < d;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f), z = v, w = v;
+        if (mine) {
+            v = *reinterpret_cast<const float4*>(o + t * o_t + c0 + c);
+            z = *reinterpret_cast<const float4*>(gate + t * gate_t + c0 + c);
+            w = *reinterpret_cast<const float4*>(weight + c0 + c);
+        }
+        float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+        for (int m = group >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+        const float f = 1.f / sqrtf(ss / (float)d + eps);
+        if (mine)
+            shift_store4(out + t * out_t + c0 + c, make_float4(v.x * f * w.x * (z.x / (1.f + expf(-z.x))), v.y * f * w.y * (z.y / (1.f + expf(-z.y))),
+                                                              v.z * f * w.z * (z.z / (1.f + expf(-z.z))), v.w * f * w.w * (z.w / (1.f + expf(-z.w)))));
+        return;
+    }
+    if (!valid) return;
     const float* y = o + t * o_t + c0;
     const float* z = gate + t * gate_t + c0;
     T* dst = out + t * out_t + c0;
     float ss = 0.f;
-    if ((d & 1) == 0 && d <= 256 && ((o_t | gate_t | out_t) & 1) == 0) {      // pairs, the row in registers
-        float2 v[4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int c = 2 * (lane + 32 * i);
-            v[i] = c < d ? *reinterpret_cast<const float2*>(y + c) : make_float2(0.f, 0.f);
-            ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, ss));
-        }
-        ss = warp_sum(ss);
-        const float f = 1.f / sqrtf(ss / (float)d + eps);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int c = 2 * (lane + 32 * i);
-            if (c < d) {
-                const float2 zz = *reinterpret_cast<const float2*>(z + c), w = *reinterpret_cast<const float2*>(weight + c0 + c);
-                const float a = v[i].x * f * w.x * (zz.x / (1.f + expf(-zz.x))), b = v[i].y * f * w.y * (zz.y / (1.f + expf(-zz.y)));
-                store2(dst + c, a, b);
-            }
-        }
-        return;
-    }
     for (int c = lane; c < d; c += 32) ss = fmaf(y[c], y[c], ss);
     ss = warp_sum(ss);
     const float f = 1.f / sqrtf(ss / (float)d + eps);
@@ -503,10 +498,15 @@ LLMP_API int llmp_wkv_gate(const float* o, long o_t, const float* gate, long gat
     if (N <= 0) return 0;
     LLMP_REQUIRE(H > 0 && d > 0, "wkv_gate: bad sizes heads=%d dim=%d", H, d);
     const long items = (long)N * H;
-    const dim3 grid((unsigned)((items + 3) / 4));
-    if (out_dtype == LLMP_BF16)
-        llmp_launch_dependent(wkv_gate_kernel<bf16>, grid, dim3(128), 0, stream, o, o_t, gate, gate_t, weight, (bf16*)out, out_t, items, H, d, eps);
-    else
-        llmp_launch_dependent(wkv_gate_kernel<float>, grid, dim3(128), 0, stream, o, o_t, gate, gate_t, weight, (float*)out, out_t, items, H, d, eps);
+    int group = 32;
+    const bool vec = d % 4 == 0 && d <= 128 && o_t % 4 == 0 && gate_t % 4 == 0 && out_t % 4 == 0 &&
+                     ((size_t)o | (size_t)gate | (size_t)weight | (size_t)out) % 16 == 0;
+    if (vec) for (group = 1; 4 * group < d;) group *= 2;
+    const dim3 grid((unsigned)((items * group + 127) / 128));
+#define LLMP_WKV_GATE(T, VEC) \
+    llmp_launch_dependent(wkv_gate_kernel<T, VEC>, grid, dim3(128), 0, stream, o, o_t, gate, gate_t, weight, (T*)out, out_t, items, H, d, group, eps)
+    if (out_dtype == LLMP_BF16) { if (vec) LLMP_WKV_GATE(bf16, true); else LLMP_WKV_GATE(bf16, false); }
+    else { if (vec) LLMP_WKV_GATE(float, true); else LLMP_WKV_GATE(float, false); }
+#undef LLMP_WKV_GATE
     return llmp_check_launch("wkv_gate");
 }

@@ -996,7 +996,7 @@ def expert_rows(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     return out
 
 
-EXPERT_TC_MIN_ROWS = 512             # pairs from which those products are the tcgen05 ones
+EXPERT_TC_MIN_ROWS = 128             # pairs from which those products are the tcgen05 ones
 EXPERT_GROUPED_MIN_ROWS = 33         # (token, choice) pairs from which a step's experts run as grouped products
 
 
@@ -1764,12 +1764,12 @@ def _wkv_rows(dim: int) -> int:
     return rows
 
 
-WKV_SEGMENT_TOKENS = 256             # tokens of a segment of a prompt whose segments run side by side
+WKV_SEGMENT_TOKENS = 128             # tokens of a segment of a prompt whose segments run side by side
 
 
 def wkv_segments(longest: int, requests: int, heads: int, dim: int) -> int:
     """Into how many segments a step cuts its requests: long portions whose blocks alone would leave most of the GPU's warps idle."""
-    if longest < 2 * WKV_SEGMENT_TOKENS or requests * heads * -(-dim // 32) >= 6 * sm_count():
+    if longest < 4 * WKV_SEGMENT_TOKENS or requests * heads * -(-dim // 32) >= 6 * sm_count():
         return 1
     return -(-longest // WKV_SEGMENT_TOKENS)
 

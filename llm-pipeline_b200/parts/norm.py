@@ -22,16 +22,21 @@ from .registry import register_norm
 class RMSNorm(Norm):
     graph_safe = True
 
-    def __init__(self, prefix: str, size: int, eps: float, offset: float = 0.0, name: Optional[str] = None, gain: float = 1.0):
+    def __init__(self, prefix: str, size: int, eps: float, offset: float = 0.0, name: Optional[str] = None, gain: float = 1.0,
+                 unused=()):
         """``offset``: the stored weight w stands for ``offset + w`` (1.0 for weights kept around zero); ``name``: the
         tensor's full name where it is not ``<prefix>.weight``; ``gain``: a constant factor on the normed rows (a layer
-        that adds ``m * norm(sublayer)`` to its residual gives that norm the gain m)."""
+        that adds ``m * norm(sublayer)`` to its residual gives that norm the gain m); ``unused``: names of further weights a
+        checkpoint may hold although nothing of this layer reads them."""
         self.prefix, self.size, self.eps, self.offset, self.gain = prefix, int(size), float(eps), float(offset), float(gain)
         self.name = name or f"{prefix}.weight"
+        self.unused = tuple(unused)
         self.weight: Optional[torch.Tensor] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {self.name: ParamSpec((self.size,), role="vector", init="small" if self.offset else "norm")}
+        specs = {self.name: ParamSpec((self.size,), role="vector", init="small" if self.offset else "norm")}
+        specs.update({name: ParamSpec((self.size,), role="vector", optional=True, init="norm") for name in self.unused})
+        return specs
 
     def load(self, get: TensorGetter) -> None:
         self.weight = get(self.name, "vector").contiguous()
