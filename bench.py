@@ -667,7 +667,7 @@ def zupilorn_work(z, tokens, keys_per_token, decode):
         work["expert_rows"] = (att_layers * pairs * expert_weights, 0.0)
     else:
         work["expert_rows"] = (0.0, att_layers * 2.0 * pairs * 3 * z["expert_ff"] * D)
-    work["expert_grouped"] = work["expert_rows"]
+    work["expert_grouped"] = work["expert_tc"] = work["expert_rows"]
     return work
 
 
@@ -803,7 +803,7 @@ def razelorn_work(z, tokens, keys_per_token, decode):
         work["expert_rows"] = (moe_layers * pairs * expert_weights, 0.0)
     else:
         work["expert_rows"] = (0.0, moe_layers * 2.0 * pairs * 3 * z["expert_ff"] * D)
-    work["expert_grouped"] = work["expert_rows"]
+    work["expert_grouped"] = work["expert_tc"] = work["expert_rows"]
     return work
 
 
@@ -978,7 +978,7 @@ def zasudra_work(z, tokens, keys_per_token, decode, requests=1):
         work["expert_rows"] = (L * pairs * 2 * z["expert_ff"] * D * 2, 0.0)
     else:
         work["expert_rows"] = (0.0, L * 2.0 * pairs * 2 * z["expert_ff"] * D)
-    work["expert_grouped"] = work["expert_rows"]
+    work["expert_grouped"] = work["expert_tc"] = work["expert_rows"]
     return work
 
 

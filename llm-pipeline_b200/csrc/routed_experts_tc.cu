@@ -140,7 +140,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
     pdl_wait();                                                  // what the kernels before wrote is complete
     pdl_trigger();
     const int m_tiles = *a.num_tiles, n_tiles = (a.cols + OUT_COLS - 1) / OUT_COLS;
-    const int total = m_tiles * n_tiles;
+    const int total = m_tiles * n_tiles;                         // in the order of the experts: what runs at one time shares rows and weights
     const int kblocks = (a.K + MT_BK - 1) / MT_BK;
     const int w_rows = (GATED ? 2 : 1) * a.cols;                 // weight rows of an expert
 
@@ -149,7 +149,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
             int it = 0;
             bool ok = true;
             for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
-                const int m = tile % m_tiles, c0 = (tile / m_tiles) * OUT_COLS;
+                const int m = tile / n_tiles, c0 = (tile % n_tiles) * OUT_COLS;
                 const int b0 = a.tile_expert[m] * w_rows + c0;
                 for (int kb = 0; kb < kblocks; ++kb, ++it) {
                     const int s = it % MT_STAGES;
@@ -169,7 +169,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
             int it = 0, n = 0;
             bool ok = true;
             for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x, ++n) {
-                const int c0 = (tile / m_tiles) * OUT_COLS;
+                const int c0 = (tile % n_tiles) * OUT_COLS;
                 // a last tile of at most half the columns takes half the product (its other weight rows are another expert's)
                 const uint32_t idesc = !GATED && a.cols - c0 <= MT_COLS / 2 ? umma_idesc(MT_ROWS, MT_COLS / 2) : umma_idesc(MT_ROWS, MT_COLS);
                 const int acc = n & 1;
@@ -194,7 +194,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__
         int n = 0;
         for (int tile = blockIdx.x; tile < total; tile += gridDim.x, ++n) {
             const int acc = n & 1;
-            const int m = tile % m_tiles, c0 = (tile / m_tiles) * OUT_COLS;
+            const int m = tile / n_tiles, c0 = (tile % n_tiles) * OUT_COLS;
             const int row = m * MT_ROWS + quarter * 32 + lane;
             const int pair = a.sorted_pair[row];
             const float w = FIRST && pair >= 0 ? a.wts[pair] : 0.f;
