@@ -9,7 +9,8 @@ from .razelorn import RazelornConfig
 from .nufolix import NufolixConfig
 from .tupidra import TupidraConfig
 from .zasudra import ZasudraConfig
+from .zavizen import ZavizenConfig
 
-__all__ = ["LayerSpec", "ModelConfig", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen3Config", "ZupilornConfig", "RazelornConfig", "NufolixConfig", "TupidraConfig", "ZasudraConfig",
+__all__ = ["LayerSpec", "ModelConfig", "ModelSpec", "PartSpec", "ScheduleEntry", "Qwen3Config", "ZupilornConfig", "RazelornConfig", "NufolixConfig", "TupidraConfig", "ZasudraConfig", "ZavizenConfig",
            "architecture_name", "load_config", "register_architecture", "resolve_config",
            "supported_architectures"]

@@ -78,6 +78,7 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     max_position: int
+    streams: Optional[int] = None           # copies of the hidden state that hyper-connections join (None: one plain residual)
 
     def validate(self) -> None:
         seen = set()

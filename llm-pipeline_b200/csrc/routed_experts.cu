@@ -2,7 +2,8 @@
 //   route_topk:      router logits in float32 (float32 copy of the router matrix, the token's row as stored); scores by
 //                    sigmoid (each logit alone) or softmax (over all router outputs); the `top` largest of
 //                    score (+ a correction per router output, if given); a chosen expert's weight is its score
-//                    without the correction. Or the `top` largest logits, and a softmax over those alone. A bias per
+//                    without the correction. The outputs may form groups of neighbours, of which only those with the largest
+//                    best entries can be chosen from; the chosen weights may be divided by their sum and scaled. Or the `top` largest logits, and a softmax over those alone. A bias per
 //                    router output joins the logits, if given. A further row of the matrix, if asked for, gives a gate per token:
 //                    sigmoid of its logit.
 //   expert_gate_up:  per (token, choice), with w the choice's weight, by the form of the expert:
@@ -35,8 +36,15 @@ __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
-// The choice of one token by one warp: `logits` [E (+ 1: the gate's)] in shared memory, overwritten; `score` [E] is scratch.
-__device__ __forceinline__ void route_choose(float* logits, float* score, int n, int top, int* __restrict__ ids, float* __restrict__ wts, int E,
+struct RouteRule {
+    int groups, keep;       // equal groups of neighbours and how many of them can be chosen from (0 groups: no such limit)
+    int normalize;          // the chosen weights are divided by (their sum + 1e-20)
+    float factor;           // and scaled
+};
+
+// The choice of one token by one warp: `logits` [E (+ 1: the gate's)] in shared memory, overwritten; `score` [E] and `best_of` [groups] are
+// scratch.
+__device__ __forceinline__ void route_choose(float* logits, float* score, float* best_of, const RouteRule& rule, int n, int top, int* __restrict__ ids, float* __restrict__ wts, int E,
                                              int mode, const float* __restrict__ correction, float* __restrict__ gate, int lane) {
     const bool softmax = mode == 1;
     if (gate && lane == 0) gate[n] = 1.f / (1.f + expf(-logits[E]));
@@ -65,6 +73,23 @@ __device__ __forceinline__ void route_choose(float* logits, float* score, int n,
         }
         __syncwarp();
     }
+    if (rule.groups > 0) {
+        const int per = E / rule.groups;
+        for (int g = lane; g < rule.groups; g += 32) {
+            float b = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, logits[e]);
+            best_of[g] = b;
+        }
+        __syncwarp();
+        for (int g = lane; g < rule.groups; g += 32) {
+            const float b = best_of[g];
+            int ahead = 0;
+            for (int o = 0; o < rule.groups; ++o) ahead += best_of[o] > b || (best_of[o] == b && o < g);
+            if (ahead >= rule.keep)
+                for (int e = g * per; e < (g + 1) * per; ++e) logits[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
     const bool by_score = softmax || correction;
     float first = 0.f, total = 0.f;                      // mode 2: the largest logit, and the sum of the chosen exponentials
     for (int k = 0; k < top; ++k) {
@@ -87,27 +112,30 @@ __device__ __forceinline__ void route_choose(float* logits, float* score, int n,
                 total += w;
             } else {
                 w = by_score ? score[at] : 1.f / (1.f + expf(-best));
+                total += w;
             }
             wts[(size_t)n * top + k] = w;
             logits[at] = -INFINITY;
         }
         __syncwarp();
     }
-    if (mode == 2) {
+    if (mode == 2 || rule.normalize || rule.factor != 1.f) {
         total = __shfl_sync(0xffffffffu, total, 0);
-        for (int k = lane; k < top; k += 32) wts[(size_t)n * top + k] /= total;
+        const float by = mode == 2 ? total : (rule.normalize ? total + 1e-20f : 1.f);
+        for (int k = lane; k < top; k += 32) wts[(size_t)n * top + k] = wts[(size_t)n * top + k] / by * rule.factor;
     }
 }
 
 __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const float* __restrict__ wr, int top, int* __restrict__ ids,
                                   float* __restrict__ wts, int Hd, int E, int mode, const float* __restrict__ bias,
-                                  const float* __restrict__ correction, float* __restrict__ gate) {
+                                  const float* __restrict__ correction, float* __restrict__ gate, const RouteRule rule) {
     pdl_wait();                                    // what the kernels before wrote is complete
     pdl_trigger();
     extern __shared__ float route_smem[];
     float* row = route_smem;                                 // [Hd]: the token's row, read once
     float* logits = row + Hd;                                // [E + 1]: logits, then what the choice goes by
     float* score = logits + E + 1;                           // [E]: softmax scores (softmax only)
+    float* best_of = score + E;                              // [groups]
     const bool vec = Hd % 8 == 0 && ((size_t)wr & 15) == 0;
     const int rows_w = gate ? E + 1 : E;                     // the gate's row follows the experts' rows
     const int n = blockIdx.x;
@@ -141,7 +169,7 @@ __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const 
         if (lane == 0) logits[e] = (bias && e < E) ? s + bias[e] : s;
     }
     __syncthreads();
-    if (warp == 0) route_choose(logits, score, n, top, ids, wts, E, mode, correction, gate, lane);
+    if (warp == 0) route_choose(logits, score, best_of, rule, n, top, ids, wts, E, mode, correction, gate, lane);
 }
 
 // The same for steps of many rows: a block takes ROUTE_TOKENS tokens, so that the router matrix is read once for all of
@@ -150,7 +178,7 @@ __global__ void route_topk_kernel(const void* __restrict__ h, int h_bf16, const 
 __global__ void __launch_bounds__(256) route_topk_tile_kernel(const void* __restrict__ h, int h_bf16, const float* __restrict__ wr, int top,
                                                               int* __restrict__ ids, float* __restrict__ wts, int N, int Hd, int E, int mode,
                                                               const float* __restrict__ bias, const float* __restrict__ correction,
-                                                              float* __restrict__ gate) {
+                                                              float* __restrict__ gate, const RouteRule rule) {
     extern __shared__ float route_smem[];
     pdl_wait();                                    // what the kernels before wrote is complete
     pdl_trigger();
@@ -158,6 +186,7 @@ __global__ void __launch_bounds__(256) route_topk_tile_kernel(const void* __rest
     float* rows = route_smem;                                // [ROUTE_TOKENS][Hd]
     float* logits = rows + ROUTE_TOKENS * Hd;                // [ROUTE_TOKENS][E + 1]
     float* score = logits + ROUTE_TOKENS * (E + 1);          // [ROUTE_TOKENS][E]
+    float* best_of = score + ROUTE_TOKENS * E;               // [ROUTE_TOKENS][groups]
     const int n0 = blockIdx.x * ROUTE_TOKENS, cnt = min(ROUTE_TOKENS, N - n0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool vec = Hd % 8 == 0 && (((size_t)h | (size_t)wr) & 15) == 0;
@@ -221,29 +250,33 @@ __global__ void __launch_bounds__(256) route_topk_tile_kernel(const void* __rest
         if (e < rows_w) logits[(lane & 7) * (E + 1) + e] = (bias && e < E) ? acc[0] + bias[e] : acc[0];
     }
     __syncthreads();
-    if (warp < cnt) route_choose(logits + warp * (E + 1), score + warp * E, n0 + warp, top, ids, wts, E, mode, correction, gate, lane);
+    if (warp < cnt) route_choose(logits + warp * (E + 1), score + warp * E, best_of + warp * rule.groups, rule, n0 + warp, top, ids, wts, E, mode, correction, gate, lane);
 }
 
 // mode: 0 sigmoid scores, 1 softmax over the E router outputs, 2 softmax over the chosen logits. bias: float32 [E] or null. correction: float32 [E] or null. gate: float32 [N] or
 // null; when given, w_router has E + 1 rows and gate[n] = sigmoid(row E . h[n]).
 LLMP_API int llmp_route_topk(const void* h, int h_dtype, const float* w_router, int top, int* ids, float* wts, int N, int Hd, int E,
-                             int mode, const float* bias, const float* correction, float* gate, cudaStream_t stream) {
+                             int mode, const float* bias, const float* correction, float* gate, int groups, int keep, int normalize, float factor,
+                             cudaStream_t stream) {
     if (N <= 0) return 0;
     LLMP_REQUIRE(mode >= 0 && mode <= 2 && (mode != 2 || !correction), "route_topk: mode %d", mode);
     LLMP_REQUIRE(E > 0 && top > 0 && top <= E && Hd > 0 && E <= 8192, "route_topk: bad sizes experts=%d top=%d width=%d", E, top, Hd);
-    const size_t smem = (size_t)(2 * E + 1 + Hd) * sizeof(float);
+    LLMP_REQUIRE(groups >= 0 && (groups == 0 || (E % groups == 0 && keep > 0 && keep <= groups && (long)keep * (E / groups) >= top)),
+                 "route_topk: %d of %d groups of %d experts for %d choices", keep, groups, E, top);
+    const RouteRule rule = {groups, keep, normalize, factor};
+    const size_t smem = (size_t)(2 * E + 1 + Hd + groups) * sizeof(float);
     LLMP_REQUIRE(smem <= 200 * 1024, "route_topk: a row of %d entries does not fit shared memory", Hd);
-    const size_t tile_smem = (size_t)ROUTE_TOKENS * (2 * E + 1 + Hd) * sizeof(float);
+    const size_t tile_smem = (size_t)ROUTE_TOKENS * (2 * E + 1 + Hd + groups) * sizeof(float);
     if (N > 64 && tile_smem <= 200 * 1024) {
         LLMP_ALLOW_SMEM(route_topk_tile_kernel, tile_smem);
         llmp_launch_dependent(route_topk_tile_kernel, dim3((N + ROUTE_TOKENS - 1) / ROUTE_TOKENS), dim3(256), tile_smem, stream, h,
-                              (int)(h_dtype == LLMP_BF16), w_router, top, ids, wts, N, Hd, E, mode, bias, correction, gate);
+                              (int)(h_dtype == LLMP_BF16), w_router, top, ids, wts, N, Hd, E, mode, bias, correction, gate, rule);
         return llmp_check_launch("route_topk");
     }
     LLMP_ALLOW_SMEM(route_topk_kernel, smem);
     // few rows (a decode step): a warp per expert, so that the router matrix is read by many warps at once
     llmp_launch_dependent(route_topk_kernel, dim3(N), dim3(N <= 64 ? 1024 : 256), smem, stream, h, (int)(h_dtype == LLMP_BF16), w_router,
-                          top, ids, wts, Hd, E, mode, bias, correction, gate);
+                          top, ids, wts, Hd, E, mode, bias, correction, gate, rule);
     return llmp_check_launch("route_topk");
 }
 

@@ -3,6 +3,8 @@
 // Per head h (group g = h / (H / G)), with x_t [P], B_t and C_t [N] of the token and S [N, P] the head's state:
 //   dt = softplus(dt_raw[t, h] + dt_bias[h]),  a = exp(-exp(A_log[h]) * dt)
 //   S <- a S + dt B_t x_t^T,   y_t = S^T C_t + D[h] x_t
+// or, with a decay that is a constant of the head (retention: B, C, x are keys, queries and values):
+//   S <- decay[h] S + B_t x_t^T,   y_t = S^T C_t                 the constant as a float and what the float leaves of it
 // Everything is float32. A block owns (request, head, a range of columns) and walks the request's tokens in order; lane
 // (p, r) holds the rows r, r + R, r + 2R .. of column p in registers, the sums over rows are shuffles. The state lives
 // in the request's slot as two copies that take turns by the parity of the last position written.
@@ -10,6 +12,7 @@
 // gated_group_norm: rows [tokens, W] cut into groups of `gs` entries.
 //   mode 0: v = y * silu(gate);  out = v / sqrt(mean_group(v^2) + eps) * weight[column]
 //   mode 1: out = y / sqrt(mean_group(y^2) + eps) * weight[column % gs] * sigmoid(gate)
+//   mode 2: out = y / sqrt(mean_group(y^2) + eps) * silu(gate)
 #include "common.cuh"
 
 namespace {
@@ -17,9 +20,11 @@ namespace {
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
 struct ScanArgs {
-    const float* xbc; long xbc_t;            // [tokens, H P + 2 G N]: x | B | C
+    const float* x; long x_t;                // [tokens, H P]
+    const float* b; const float* c; long bc_t;   // [tokens, G N] each
     const float* dt; long dt_t;              // [tokens, >= H]
     const float* dt_bias; const float* a_log; const float* d_skip;    // [H]
+    const float* decay;                      // [2][H]: constants and what their float leaves of them, or null
     float* state; long state_slot; long state_half;                   // copy: [H][N][P]
     const int* q_start; const int* slots; const int* positions;
     float* y; long y_t;                      // [tokens, H P]
@@ -59,7 +64,7 @@ template <int V> __device__ __forceinline__ SsVec<V> ss_load(const float* p) {
 // through a ring of SS_STAGES stages of `stage_tokens` tokens (cp.async, 16 bytes where the rows allow it), a token
 // each in turn, and the first of them turns each token's raw step size into (dt, decay) before the stage's barrier:
 // one barrier per stage, not per token.
-template <int NT, int R>
+template <int NT, int R, bool FIXED>
 __global__ void __launch_bounds__(SS_THREADS + 32 * SS_COPY_WARPS) ssd_scan_kernel(const ScanArgs a, const int stage_tokens, const int vec) {
     extern __shared__ __align__(16) float smem[];
     constexpr int V = NT < 4 ? NT : 4;
@@ -89,8 +94,9 @@ __global__ void __launch_bounds__(SS_THREADS + 32 * SS_COPY_WARPS) ssd_scan_kern
     }
     for (int i = threadIdx.x; i < SS_STAGES * stage_tokens * ROW; i += blockDim.x) smem[i] = 0.f;
     __syncthreads();
-    const float neg_a = -expf(a.a_log[h]), bias = a.dt_bias[h], skip = a.d_skip[h];
-    const size_t x_at = (size_t)h * P, b_at = (size_t)a.H * P + (size_t)g * N, c_at = b_at + (size_t)a.G * N;
+    const float neg_a = FIXED ? 0.f : -expf(a.a_log[h]), bias = FIXED ? 0.f : a.dt_bias[h], skip = FIXED ? 0.f : a.d_skip[h];
+    const float fixed_hi = FIXED ? a.decay[h] : 0.f, fixed_lo = FIXED ? a.decay[a.H + h] : 0.f;
+    const size_t x_at = (size_t)h * P, bc_at = (size_t)g * N;
     const int ncols = min(COLS, P - j0);
     const int stages = (end - begin + stage_tokens - 1) / stage_tokens;
     auto issue = [&](int s) {                           // the copying warp only
@@ -99,11 +105,11 @@ __global__ void __launch_bounds__(SS_THREADS + 32 * SS_COPY_WARPS) ssd_scan_kern
             const int t0 = begin + s * stage_tokens;
             const int cnt = min(stage_tokens, end - t0);
             for (int tt = copy_warp; tt < cnt; tt += SS_COPY_WARPS) {
-                const float* src = a.xbc + (size_t)(t0 + tt) * a.xbc_t;
+                const size_t t = (size_t)(t0 + tt);
                 float* dst = dst0 + (size_t)tt * ROW;
-                ss_copy_row(dst, src + b_at, N, vec & 1, lane);
-                ss_copy_row(dst + NP, src + c_at, N, vec & 1, lane);
-                ss_copy_row(dst + 2 * NP, src + x_at + j0, ncols, vec & 2, lane);
+                ss_copy_row(dst, a.b + t * a.bc_t + bc_at, N, vec & 1, lane);
+                ss_copy_row(dst + NP, a.c + t * a.bc_t + bc_at, N, vec & 1, lane);
+                ss_copy_row(dst + 2 * NP, a.x + t * a.x_t + x_at + j0, ncols, vec & 2, lane);
             }
         }
         asm volatile("cp.async.commit_group;\n" ::: "memory");
@@ -114,7 +120,7 @@ __global__ void __launch_bounds__(SS_THREADS + 32 * SS_COPY_WARPS) ssd_scan_kern
         const int t0 = begin + s * stage_tokens;
         const int cnt = min(stage_tokens, end - t0);
         if (loader) {
-            for (int tt = lane; tt < cnt && copy_warp == 0; tt += 32) {   // step sizes and decays of the stage's tokens
+            for (int tt = lane; tt < cnt && copy_warp == 0 && !FIXED; tt += 32) {   // step sizes and decays of the stage's tokens
                 const float dt = softplus_f(a.dt[(size_t)(t0 + tt) * a.dt_t + h] + bias);
                 base[(size_t)tt * ROW + 2 * NP + COLS] = dt;
                 base[(size_t)tt * ROW + 2 * NP + COLS + 1] = expf(neg_a * dt);
@@ -128,9 +134,9 @@ __global__ void __launch_bounds__(SS_THREADS + 32 * SS_COPY_WARPS) ssd_scan_kern
         }
         for (int tt = 0; tt < cnt; ++tt) {
             const float* cur = base + (size_t)tt * ROW;
-            const float dt = cur[2 * NP + COLS], decay = cur[2 * NP + COLS + 1];
+            const float decay = FIXED ? fixed_hi : cur[2 * NP + COLS + 1];
             const float xv = cur[2 * NP + col];
-            const float dx = dt * xv;
+            const float dx = FIXED ? xv : cur[2 * NP + COLS] * xv;
             float y[2] = {0.f, 0.f};
 #pragma unroll
             for (int i4 = 0; i4 < NT / V; ++i4) {
@@ -139,14 +145,16 @@ __global__ void __launch_bounds__(SS_THREADS + 32 * SS_COPY_WARPS) ssd_scan_kern
 #pragma unroll
                 for (int e = 0; e < V; ++e) {
                     const int i = i4 * V + e;
-                    S[i] = fmaf(decay, S[i], bb.v[e] * dx);
+                    float add = bb.v[e] * dx;
+                    if constexpr (FIXED) add = fmaf(fixed_lo, S[i], add);
+                    S[i] = fmaf(decay, S[i], add);
                     y[e & 1] = fmaf(S[i], cc.v[e], y[e & 1]);
                 }
             }
             float ys = y[0] + y[1];
 #pragma unroll
             for (int m = R >> 1; m > 0; m >>= 1) ys += __shfl_xor_sync(0xffffffffu, ys, m);
-            if (rr == 0 && valid) a.y[(size_t)(t0 + tt) * a.y_t + x_at + p] = fmaf(skip, xv, ys);
+            if (rr == 0 && valid) a.y[(size_t)(t0 + tt) * a.y_t + x_at + p] = FIXED ? ys : fmaf(skip, xv, ys);
         }
     }
     if (loader) asm volatile("cp.async.wait_group 0;\n" ::: "memory");
@@ -189,25 +197,20 @@ __global__ void gated_group_norm_kernel(const NormArgs a) {
         float v = y[i];
         const float z = gate[i];
         if (a.mode == 0) v = v * (z / (1.f + expf(-z))) * inv * a.weight[c0 + i];
-        else v = v * inv * a.weight[i] * (1.f / (1.f + expf(-z)));
+        else v = v * inv * (a.mode == 1 ? a.weight[i] : z) * (1.f / (1.f + expf(-z)));
         out[i] = from_float<T>(v);
     }
 }
 
 }  // namespace
 
-LLMP_API int llmp_ssd_scan(const float* xbc, long xbc_t, const float* dt, long dt_t, const float* dt_bias, const float* a_log,
-                           const float* d_skip, float* state, long state_slot, long state_half, const int* q_start,
-                           const int* slots, const int* positions, float* y, long y_t, int R, int H, int G, int N, int P,
-                           cudaStream_t stream) {
+static int launch_scan(const ScanArgs& a, int R, cudaStream_t stream) {
+    const int H = a.H, G = a.G, N = a.N, P = a.P;
+    const bool fixed = a.decay != nullptr;
     if (R <= 0) return 0;
     LLMP_REQUIRE(H > 0 && G > 0 && H % G == 0 && N > 0 && P > 0 && P <= 1024, "ssd_scan: bad sizes heads=%d groups=%d state=%d vdim=%d",
                  H, G, N, P);
     LLMP_REQUIRE(H <= 65535 && (P + 3) / 4 <= 65535, "ssd_scan: too many heads %d or columns %d", H, P);
-    ScanArgs a;
-    a.xbc = xbc; a.xbc_t = xbc_t; a.dt = dt; a.dt_t = dt_t; a.dt_bias = dt_bias; a.a_log = a_log; a.d_skip = d_skip;
-    a.state = state; a.state_slot = state_slot; a.state_half = state_half; a.q_start = q_start; a.slots = slots;
-    a.positions = positions; a.y = y; a.y_t = y_t; a.H = H; a.G = G; a.N = N; a.P = P;
     // lanes that share a column: the fewest (a power of two up to 32) that leave a lane at most 16 rows (32 past 512 rows)
     int rows = 1;
     while (rows < 32 && (N + rows - 1) / rows > 16) rows *= 2;
@@ -223,15 +226,18 @@ LLMP_API int llmp_ssd_scan(const float* xbc, long xbc_t, const float* dt, long d
     const size_t smem = SS_STAGES * stage_tokens * row_bytes;
     LLMP_REQUIRE(smem <= 200 * 1024, "ssd_scan: state size %d does not fit shared memory", N);
     int vec = 0;
-    if (((uintptr_t)xbc & 15) == 0 && xbc_t % 4 == 0 && P % 4 == 0) {
-        if (N % 4 == 0 && ((long)H * P) % 4 == 0) vec |= 1;
-        if ((nt * rows) % 4 == 0) vec |= 2;     // the columns' place in a row of the ring is 16-byte aligned
-    }
+    if ((((uintptr_t)a.b | (uintptr_t)a.c) & 15) == 0 && a.bc_t % 4 == 0 && N % 4 == 0) vec |= 1;
+    if (((uintptr_t)a.x & 15) == 0 && a.x_t % 4 == 0 && P % 4 == 0 && (nt * rows) % 4 == 0) vec |= 2;   // and the columns' place in a row of the ring
     dim3 grid(R, H, (P + cols - 1) / cols);
 #define LLMP_SCAN(NT, RW)                                                                         \
     if (nt == NT && rows == RW) {                                                                 \
-        LLMP_ALLOW_SMEM((ssd_scan_kernel<NT, RW>), smem);                                         \
-        ssd_scan_kernel<NT, RW><<<grid, SS_THREADS + 32 * SS_COPY_WARPS, smem, stream>>>(a, stage_tokens, vec);   \
+        if (fixed) {                                                                              \
+            LLMP_ALLOW_SMEM((ssd_scan_kernel<NT, RW, true>), smem);                               \
+            ssd_scan_kernel<NT, RW, true><<<grid, SS_THREADS + 32 * SS_COPY_WARPS, smem, stream>>>(a, stage_tokens, vec);    \
+        } else {                                                                                  \
+            LLMP_ALLOW_SMEM((ssd_scan_kernel<NT, RW, false>), smem);                              \
+            ssd_scan_kernel<NT, RW, false><<<grid, SS_THREADS + 32 * SS_COPY_WARPS, smem, stream>>>(a, stage_tokens, vec);   \
+        }                                                                                         \
     } else
     LLMP_SCAN(1, 1) LLMP_SCAN(2, 1) LLMP_SCAN(4, 1) LLMP_SCAN(8, 1) LLMP_SCAN(16, 1) LLMP_SCAN(16, 2) LLMP_SCAN(16, 4)
     LLMP_SCAN(16, 8) LLMP_SCAN(16, 16) LLMP_SCAN(16, 32) LLMP_SCAN(32, 32)
@@ -243,11 +249,34 @@ LLMP_API int llmp_ssd_scan(const float* xbc, long xbc_t, const float* dt, long d
     return llmp_check_launch("ssd_scan");
 }
 
+LLMP_API int llmp_ssd_scan(const float* xbc, long xbc_t, const float* dt, long dt_t, const float* dt_bias, const float* a_log,
+                           const float* d_skip, float* state, long state_slot, long state_half, const int* q_start,
+                           const int* slots, const int* positions, float* y, long y_t, int R, int H, int G, int N, int P,
+                           cudaStream_t stream) {
+    ScanArgs a = {};
+    a.x = xbc; a.x_t = xbc_t; a.b = xbc + (size_t)H * P; a.c = a.b + (size_t)G * N; a.bc_t = xbc_t;
+    a.dt = dt; a.dt_t = dt_t; a.dt_bias = dt_bias; a.a_log = a_log; a.d_skip = d_skip;
+    a.state = state; a.state_slot = state_slot; a.state_half = state_half; a.q_start = q_start; a.slots = slots;
+    a.positions = positions; a.y = y; a.y_t = y_t; a.H = H; a.G = G; a.N = N; a.P = P;
+    return launch_scan(a, R, stream);
+}
+
+// q, k [tokens, H N] and v [tokens, H P] with one stride; decay [2][H].
+LLMP_API int llmp_retention_scan(const float* q, const float* k, const float* v, long qkv_t, const float* decay, float* state,
+                                 long state_slot, long state_half, const int* q_start, const int* slots, const int* positions,
+                                 float* y, long y_t, int R, int H, int N, int P, cudaStream_t stream) {
+    ScanArgs a = {};
+    a.x = v; a.x_t = qkv_t; a.b = k; a.c = q; a.bc_t = qkv_t; a.decay = decay;
+    a.state = state; a.state_slot = state_slot; a.state_half = state_half; a.q_start = q_start; a.slots = slots;
+    a.positions = positions; a.y = y; a.y_t = y_t; a.H = H; a.G = H; a.N = N; a.P = P;
+    return launch_scan(a, R, stream);
+}
+
 LLMP_API int llmp_gated_group_norm(const float* y, long y_t, const float* gate, long gate_t, const float* weight, void* out,
                                    int out_dtype, long out_t, int tokens, int W, int gs, int mode, float eps,
                                    cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    LLMP_REQUIRE(W > 0 && gs > 0 && W % gs == 0 && (mode == 0 || mode == 1), "gated_group_norm: %d entries in groups of %d, mode %d",
+    LLMP_REQUIRE(W > 0 && gs > 0 && W % gs == 0 && mode >= 0 && mode <= 2, "gated_group_norm: %d entries in groups of %d, mode %d",
                  W, gs, mode);
     NormArgs a;
     a.y = y; a.y_t = y_t; a.gate = gate; a.gate_t = gate_t; a.weight = weight; a.out = out; a.out_t = out_t;

@@ -21,7 +21,7 @@ import torch
 from ..cache import CacheManager
 from ..models.model import Model
 from ..ops import kernels, timing
-from ..parts import LayerCache, ResidualStream
+from ..parts import LayerCache
 from .context import StepContext, StepShape
 
 
@@ -445,11 +445,11 @@ class ModelRunner:
             if not capturable:
                 continue
             if k > 0:
-                piece.inlet = torch.empty((ctx.num_tokens, model.spec.hidden_size), dtype=torch.float32, device=self.device)
+                piece.inlet = torch.empty(model.settled_shape(ctx.num_tokens), dtype=torch.float32, device=self.device)
             torch.cuda.synchronize(self.device)
             piece.graph = torch.cuda.CUDAGraph()
             with torch.cuda.graph(piece.graph, pool=pool):
-                stream = model.begin(ctx, self._views) if k == 0 else ResidualStream(piece.inlet, slot.history)
+                stream = model.begin(ctx, self._views) if k == 0 else model.stream_of(piece.inlet, slot.history)
                 if k == 0:
                     slot.history = stream.history        # layer results that a model with a depth mix keeps: one buffer for all pieces
                 model.run_layers(ctx, self._views, stream, first, end)
@@ -472,7 +472,7 @@ class ModelRunner:
             # eager layers: the step's arrays are the captured step's; what the layers note for themselves is not kept
             eager = copy.copy(ctx)
             eager.memo = {}
-            stream = ResidualStream(residual, slot.history)
+            stream = model.stream_of(residual, slot.history)
             model.run_layers(eager, self._views, stream, piece.first, piece.end)
             residual = stream.settle()
         slot.logits = slot.pieces[-1].outlet

@@ -14,7 +14,7 @@ from ..cache.spec import PagesSpec, StateSpec
 from ..config.base import ModelSpec, PartSpec
 from ..ops.linear import begin_step
 from ..ops.timing import nvtx_range
-from ..parts import LayerCache, ResidualStream, lookup
+from ..parts import HyperStream, LayerCache, ResidualStream, lookup
 from ..weights.source import (ParamSpec, TiedWeightError, WeightSource, check_names_and_shapes,
                               stored_dtype_policy)
 
@@ -152,7 +152,18 @@ class Model:
             if self.history_slots:
                 history = torch.empty((self.history_slots,) + tuple(residual.shape), dtype=torch.float32, device=residual.device)
                 history[0].copy_(residual)
-            return ResidualStream(residual, history)
+            return self.stream_of(residual, history)
+
+    def stream_of(self, residual: torch.Tensor, history: Optional[torch.Tensor] = None) -> ResidualStream:
+        """A stream that goes on from ``residual``: the embedding's rows, or what ``settle()`` gave."""
+        if self.spec.streams is not None:
+            return HyperStream(residual, self.spec.streams)
+        return ResidualStream(residual, history)
+
+    def settled_shape(self, tokens: int) -> Tuple[int, ...]:
+        """The shape of what ``settle()`` gives for this many tokens."""
+        H = self.spec.hidden_size
+        return (tokens, H) if self.spec.streams is None else (tokens, self.spec.streams, H)
 
     def run_layers(self, ctx, caches, stream: ResidualStream, first: int, end: int) -> None:
         """The scheduled executions first .. end - 1 on ``stream``."""

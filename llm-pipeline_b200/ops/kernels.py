@@ -79,7 +79,7 @@ _SIGNATURES = {
     "llmp_gated_act": [_P, _I, _L, _P, _I, _L, _I, _I, _P],
     "llmp_sigmoid_gate": [_P, _P, _L, _P, _I, _L, _I, _P],
     "llmp_convert_rows": [_P, _L, _P, _I, _L, _I, _P],
-    "llmp_route_topk": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P, _P],
+    "llmp_route_topk": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P, _I, _I, _I, _F, _P],
     "llmp_expert_grouped": [_P, _P, _P, _P, _P, _F, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "llmp_expert_tc": [_P, _P, _P, _P, _P, _F, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "llmp_expert_rows": [_P, _P, _P, _I, _P, _P, _F, _P, _P, _I, _I, _I, _I, _I, _I, _P],
@@ -92,6 +92,9 @@ _SIGNATURES = {
                                 _I, _I, _I, _P, _P, _P],
     "llmp_short_conv": [_P, _L, _P, _I, _P, _I, _P, _L, _L, _P, _P, _P, _P, _P, _L, _P, _I, _L, _L, _I, _I, _I, _I, _I, _I, _I, _P],
     "llmp_ssd_scan": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P],
+    "llmp_retention_scan": [_P, _P, _P, _L, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P],
+    "llmp_rotate_heads": [_P, _L, _P, _P, _I, _I, _I, _I, _F, _I, _P],
+    "llmp_stream_step": [_P, _L, _L, _P, _P, _I, _P, _F, _F, _P, _I, _P, _F, _F, _P, _P, _P, _P, _P, _I, _F, _P, _I, _P, _I, _I, _I, _P],
     "llmp_gated_group_norm": [_P, _L, _P, _L, _P, _P, _I, _L, _I, _I, _I, _I, _F, _P],
     "llmp_delta_prep": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _P],
     "llmp_delta_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P],
@@ -949,11 +952,14 @@ ROUTER_SCORES = {"sigmoid": 0, "softmax": 1, "chosen_softmax": 2}
 
 def route_topk(h: torch.Tensor, w_router: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor, *,
                softmax: bool = False, score: Optional[str] = None, bias: Optional[torch.Tensor] = None,
-               correction: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+               correction: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, groups: int = 0, keep: int = 0,
+               normalize: bool = False, factor: float = 1.0) -> None:
     """ids[n, :], weights[n, :] = the ``top`` router outputs with the largest score (+ ``correction``, if given) and their
     scores without the correction; float32 logits (+ ``bias``). The score is sigmoid(logit), or the softmax over all router
     outputs (``score`` "softmax", or ``softmax`` set); "chosen_softmax": the ``top`` largest logits, and the softmax over
-    those. With ``gate`` (float32 [tokens]) the matrix has one row more than router outputs, and
+    those. ``groups``: the router outputs form that many equal groups of neighbours, and only the ``keep`` groups whose best
+    entries are the largest can be chosen from. ``normalize``: the chosen weights are divided by (their sum + 1e-20);
+    ``factor``: and scaled. With ``gate`` (float32 [tokens]) the matrix has one row more than router outputs, and
     gate[n] = sigmoid(that row . h[n])."""
     N, Hd = h.shape
     E = w_router.shape[0] - (1 if gate is not None else 0)
@@ -969,7 +975,8 @@ def route_topk(h: torch.Tensor, w_router: torch.Tensor, top: int, ids: torch.Ten
     if gate is not None:
         _need(gate.dtype == torch.float32 and gate.is_contiguous() and gate.numel() == N, "the gate must be float32 [tokens]")
     _call("llmp_route_topk", _ptr(h), dtype_code(h.dtype), _ptr(w_router), int(top), _ptr(ids), _ptr(weights), N, Hd, E,
-          ROUTER_SCORES[score or ("softmax" if softmax else "sigmoid")], _ptr(bias), _ptr(correction), _ptr(gate), _stream())
+          ROUTER_SCORES[score or ("softmax" if softmax else "sigmoid")], _ptr(bias), _ptr(correction), _ptr(gate),
+          int(groups), int(keep), 1 if normalize else 0, float(factor), _stream())
 
 
 EXPERT_FORMS = {"clamped": 0, "silu": 1, "relu_squared": 2}     # csrc/routed_experts.cu: expert_act
@@ -1332,19 +1339,90 @@ def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: 
     return y
 
 
-def gated_group_norm(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, group_size: int, eps: float,
+def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, state_offset: int,
+                   q_start: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor, y: torch.Tensor, heads: int, dim: int,
+                   vdim: int) -> torch.Tensor:
+    """S <- decay[h] S + k_t v_t^T, y_t = S^T q_t per head (csrc/state_space.cu): ``q``, ``k`` float32 [tokens, heads dim] and ``v``
+    [tokens, heads vdim], views with one stride between tokens; ``decay`` float32 [2, heads], the constants and what their
+    float leaves of them; ``y`` float32 [tokens, heads vdim]. The state piece holds two copies of [heads, dim, vdim]."""
+    N = q.shape[0]
+    _need(all(t.dtype == torch.float32 and t.stride(1) == 1 for t in (q, k, v, y)), "retention_scan takes and gives float32 rows")
+    _need(q.shape == k.shape == (N, heads * dim) and v.shape == y.shape == (N, heads * vdim) and q.stride(0) == k.stride(0) == v.stride(0),
+          "retention_scan: rows have the wrong shape")
+    _need(decay.dtype == torch.float32 and decay.is_contiguous() and decay.shape == (2, heads), "retention_scan: decays must be float32 [2, heads]")
+    for t, name in ((q_start, "q_start"), (slots, "slots"), (positions, "positions")):
+        _i32(t, name)
+    ptr, slot_stride, half = _state_views(state, state_offset, heads * dim * vdim, "retention_scan")
+    _call("llmp_retention_scan", _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), ptr, slot_stride, half, _ptr(q_start), _ptr(slots),
+          _ptr(positions), _ptr(y), y.stride(0), slots.numel(), heads, dim, vdim, _stream())
+    return y
+
+
+def rotate_heads(x: torch.Tensor, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot: int, heads: int, scaled_from: int,
+                 dim: int, factor: float) -> torch.Tensor:
+    """In place on float32 rows of ``heads`` heads: entry i of the first ``rot`` of every head turns with entry i + rot / 2, and
+    the heads from ``scaled_from`` on are multiplied by ``factor`` afterwards."""
+    N = x.shape[0]
+    _need(x.dtype == torch.float32 and x.stride(1) == 1 and x.shape == (N, heads * dim), "rotate_heads takes float32 rows")
+    _need(rot == 0 or (cos.dtype == sin.dtype == torch.float32 and cos.is_contiguous() and sin.is_contiguous() and
+                       cos.shape == sin.shape == (N, rot // 2)), "rotate_heads: rotary tables have the wrong shape")
+    _call("llmp_rotate_heads", _ptr(x), x.stride(0), _ptr(cos), _ptr(sin), int(rot), int(heads), int(scaled_from), int(dim), float(factor), N,
+          _stream())
+    return x
+
+
+HYPER_MAX_STREAMS = 16
+
+
+def stream_step(src: torch.Tensor, streams: int, *, dst: Optional[torch.Tensor] = None, addends=(), scale: Optional[torch.Tensor] = None,
+                mix: Optional[torch.Tensor] = None, out_weights: Optional[torch.Tensor] = None, in_weights: Optional[torch.Tensor] = None,
+                weight: Optional[torch.Tensor] = None, eps: float = 0.0, out: Optional[torch.Tensor] = None,
+                rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """What lies between two sublayers joined by hyper-connections (csrc/hyper_connections.cu). ``src`` float32 [tokens, streams,
+    width], or [tokens, width] while all streams are equal. ``addends``: up to two (tensor [tokens, width], norm weight or
+    None, its eps, factor), whose sum times ``scale`` [width] is y; with ``mix`` [streams, streams] (from, to) and
+    ``out_weights`` [streams] the streams become ``sum_s mix[s, t] x_s + out[t] y``, written to ``dst`` [tokens, streams,
+    width] (may be ``src``). ``out`` = rms_norm(sum_s in[s] x_s) * ``weight`` (without ``in_weights``: the plain sum; without
+    ``weight``: not normed), of the chosen ``rows`` only if given (nothing else is written then)."""
+    T, H, S = src.shape[0], src.shape[-1], int(streams)
+    spread = src.dim() == 3
+    _need(src.dtype == torch.float32 and src.is_contiguous() and (not spread or src.shape[1] == S), "streams must be float32 [tokens, streams, width]")
+    _need(dst is None or (dst.dtype == torch.float32 and dst.is_contiguous() and tuple(dst.shape) == (T, S, H)), "stream_step: bad destination")
+    _need(len(addends) <= 2 and (not addends or mix is not None), "stream_step adds at most two addends, with a mix")
+    M = rows.numel() if rows is not None else T
+    floats = [(mix, S * S), (out_weights, S), (in_weights, S), (scale, H)]
+    args = []
+    for j in range(2):
+        y, norm, norm_eps, factor = addends[j] if j < len(addends) else (None, None, 0.0, 0.0)
+        _need(y is None or (y.is_contiguous() and tuple(y.shape) == (T, H)), "stream_step: an addend has the wrong shape")
+        floats.append((norm, H))
+        args += [_ptr(y), dtype_code(y.dtype) if y is not None else F32, _ptr(norm), float(norm_eps), float(factor)]
+    for t, n in floats:
+        _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n), "stream_step: a weight has the wrong type or size")
+    _need(out is None or (out.is_contiguous() and tuple(out.shape) == (M, H) and (weight is None or (weight.numel() == H and weight.is_contiguous()))),
+          "stream_step: output or norm weight has the wrong shape")
+    if rows is not None:
+        _i32(rows, "rows")
+    _call("llmp_stream_step", _ptr(src), S * H if spread else H, H if spread else 0, _ptr(dst), *args, _ptr(scale), _ptr(mix), _ptr(out_weights),
+          _ptr(in_weights), _ptr(weight), dtype_code(weight.dtype) if weight is not None else F32, float(eps), _ptr(out),
+          dtype_code(out.dtype) if out is not None else F32, _ptr(rows), M, S, H, _stream())
+    return out
+
+
+def gated_group_norm(y: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], out: torch.Tensor, group_size: int, eps: float,
                      gate_first: bool) -> torch.Tensor:
     """Rows cut into groups of ``group_size`` entries, each divided by its own root mean square. ``gate_first``: out =
-    rms(y silu(gate)) * weight[column]; else out = rms(y) * weight[column within the group] * sigmoid(gate). ``y`` and
-    ``gate`` float32 views, ``weight`` float32."""
+    rms(y silu(gate)) * weight[column]; else out = rms(y) * weight[column within the group] * sigmoid(gate), or, without a
+    weight, rms(y) * silu(gate). ``y`` and ``gate`` float32 views, ``weight`` float32."""
     N, W = y.shape
     _need(y.dtype == torch.float32 and gate.dtype == torch.float32 and y.stride(1) == 1 and gate.stride(1) == 1 and gate.shape == (N, W),
           "gated_group_norm takes float32 rows and gates")
-    _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == (W if gate_first else group_size),
+    _need((weight is None and not gate_first) or
+          (weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == (W if gate_first else group_size)),
           "gated_group_norm: the weight has the wrong size")
     _need(out.shape == (N, W) and out.stride(1) == 1, "gated_group_norm: the output has the wrong shape")
     _call("llmp_gated_group_norm", _ptr(y), y.stride(0), _ptr(gate), gate.stride(0), _ptr(weight), _ptr(out), dtype_code(out.dtype),
-          out.stride(0), N, W, int(group_size), 0 if gate_first else 1, float(eps), _stream())
+          out.stride(0), N, W, int(group_size), 0 if gate_first else (1 if weight is not None else 2), float(eps), _stream())
     return out
 
 

@@ -48,6 +48,18 @@ class LayerCache:
     writes: bool = True
 
 
+@dataclass
+class Addend:
+    """What a sublayer leaves to be added: ``rows`` [tokens, hidden], times ``factor``, after an RMS norm by ``weight`` (with
+    ``eps``) if it has one. A mixer or feed-forward may offer ``forward_addends(...)`` and return up to two of them whose sum is
+    its result; a block that can hand them on (``hyper_connected``) leaves norms and sums to the kernel that adds."""
+
+    rows: torch.Tensor
+    weight: Optional[torch.Tensor] = None
+    eps: float = 0.0
+    factor: float = 1.0
+
+
 class ResidualStream:
     """The hidden state between parts: a float32 residual ``[tokens, hidden]`` and a pending
     addend (with an optional bias vector) that the next norm folds in.

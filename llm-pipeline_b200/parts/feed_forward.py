@@ -20,9 +20,12 @@ from .registry import register_feed_forward
 class SwiGLU(FeedForward):
     graph_safe = True
 
-    def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, names: Optional[Dict[str, str]] = None):
+    def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, names: Optional[Dict[str, str]] = None,
+                 float32_out: bool = False):
         """``names``: the three matrices' names below ``prefix`` where they are not ``gate_proj.weight``, ``up_proj.weight``
-        and ``down_proj.weight`` (keys ``gate``, ``up``, ``down``)."""
+        and ``down_proj.weight`` (keys ``gate``, ``up``, ``down``). ``float32_out``: the last product leaves float32 (for a
+        block that takes no pending product)."""
+        self.float32_out = bool(float32_out)
         self.prefix, self.hidden_size, self.intermediate_size = prefix, int(hidden_size), int(intermediate_size)
         self.names = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
         self.names.update(names or {})
@@ -40,16 +43,21 @@ class SwiGLU(FeedForward):
     takes_scaled_rows = True             # x goes straight into gate_up_swiglu() or linear()
 
     def forward(self, x, ctx):
+        if self.float32_out:
+            return linear(self._activation(x), self.w_down, out_dtype=torch.float32), None
         out, bias = self.forward_deferred(x, ctx)
         return (out.value() if isinstance(out, PendingProduct) else out), bias
 
     def forward_deferred(self, x, ctx):
+        return pending_product(self._activation(x), self.w_down), None
+
+    def _activation(self, x):
         act = gate_up_swiglu(x, self.w_gate_up)          # the few rows of a decode step: product and activation in one kernel
         if act is None:
             gate_up = linear(x, self.w_gate_up)
             act = torch.empty((x.shape[0], self.intermediate_size), dtype=x.dtype, device=x.device)
             kernels.swiglu(gate_up, act)
-        return pending_product(act, self.w_down), None
+        return act
 
 
 @register_feed_forward("poly_norm_mlp")

@@ -12,7 +12,7 @@ before any angle is taken: with wavelength l = 2 pi / f, f stays where l < origi
 l > original / low, and between the two is the blend (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
 The frequencies are computed in float64 on the host and stored as float32; angles are float32 products.
 
-A rule with ``"kind": "ramp"`` (``factor``, ``original``, ``fast``, ``slow``) blends by the entry's index instead: with
+A rule with ``"kind": "linear"`` (``factor``) divides every frequency by the factor. One with ``"kind": "ramp"`` (``factor``, ``original``, ``fast``, ``slow``) blends by the entry's index instead: with
 ``where(t) = dims * ln(original / (2 pi t)) / (2 ln theta)`` (the index whose wave makes t turns over the original length),
 lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), dims - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1),
 the frequency is ``f_i / factor * ramp_i + f_i * (1 - ramp_i)``. A design that also scales cos and sin (by
@@ -44,7 +44,8 @@ class RotaryPositions(PositionEncoding):
             exponent = torch.arange(0, self.rotary_dim, 2, dtype=torch.int64).float() / self.rotary_dim
             self._inv_freq_cpu = 1.0 / (self.theta ** exponent)
         else:
-            rule = self.ramp_frequencies if self.frequency_scaling.get("kind") == "ramp" else self.rescaled_frequencies
+            rule = {"ramp": self.ramp_frequencies, "linear": self.divided_frequencies}.get(self.frequency_scaling.get("kind"),
+                                                                                             self.rescaled_frequencies)
             self._inv_freq_cpu = torch.tensor(rule(self.rotary_dim, self.theta, self.frequency_scaling), dtype=torch.float64).float()
         self._inv_freq = None
 
@@ -65,6 +66,13 @@ class RotaryPositions(PositionEncoding):
                 s = (original / wave - low) / (high - low)
                 out.append((1.0 - s) * f / factor + s * f)
         return out
+
+    @staticmethod
+    def divided_frequencies(rotary_dim: int, theta: float, rule: Dict[str, float]):
+        factor = float(rule["factor"])
+        if not factor > 0:
+            raise ValueError(f"a linear frequency scaling needs a positive factor, got {factor}")
+        return [theta ** (-2.0 * j / rotary_dim) / factor for j in range(rotary_dim // 2)]
 
     @staticmethod
     def ramp_frequencies(rotary_dim: int, theta: float, rule: Dict[str, float]):

@@ -3,24 +3,29 @@
 ``side_by_side`` builds its two members from part specifications (kind, sizes, tensor-name prefix below its own), so
 any two registered mixers can stand beside each other. What they ask of the cache manager is put together: at most one
 member may keep pages (the layer has one page group), and the members' states lie one after the other in the request's
-state vector, each member seeing its own column range. The sum ``left_scale * left + right_scale * right`` is float32."""
+state vector, each member seeing its own column range. The sum ``left_scale * left + right_scale * right`` is float32. With
+``out_norm_eps`` each member's result first passes an RMS norm over its row with a weight of its own (``out_norms``: the two
+names); a block that takes addends gets both results with their norms and leaves the work to the kernel that adds them."""
 
 from __future__ import annotations
 
-from typing import Any, Dict, Optional
+from typing import Any, Dict, List, Optional, Sequence
 
 import torch
 
 from ..cache.spec import StateSpec
 from ..ops import kernels
-from .base import LayerCache, Mixer, TensorGetter
+from ..weights.source import ParamSpec
+from .base import Addend, LayerCache, Mixer, TensorGetter
 from .registry import lookup, register_mixer
 
 
 @register_mixer("side_by_side")
 class SideBySide(Mixer):
-    def __init__(self, prefix: str, left: Dict[str, Any], right: Dict[str, Any], left_scale: float = 1.0, right_scale: float = 1.0):
-        """``left`` / ``right``: {"kind": a registered mixer, "args": its sizes, "prefix": its tensors' prefix below this one's}."""
+    def __init__(self, prefix: str, left: Dict[str, Any], right: Dict[str, Any], left_scale: float = 1.0, right_scale: float = 1.0,
+                 out_norm_eps: Optional[float] = None, out_norms: Sequence[str] = (), hidden_size: int = 0):
+        """``left`` / ``right``: {"kind": a registered mixer, "args": its sizes, "prefix": its tensors' prefix below this one's}. ``out_norms``: the full names of
+        the norms' weights, of ``hidden_size`` entries."""
         self.prefix = prefix
         self.scales = (float(left_scale), float(right_scale))
         self.members = tuple(lookup("mixer", m["kind"])(f"{prefix}.{m['prefix']}" if m.get("prefix") else prefix, **m["args"])
@@ -40,6 +45,11 @@ class SideBySide(Mixer):
             self._state_at.append((at, at + spec.shape[0]))
             at += spec.shape[0]
         self._state_entries = at
+        self.out_norm_eps = None if out_norm_eps is None else float(out_norm_eps)
+        self.out_norms, self.hidden_size = tuple(out_norms), int(hidden_size)
+        if (self.out_norm_eps is not None) != (len(self.out_norms) == 2 and self.hidden_size > 0):
+            raise ValueError("norms on the members' results need an eps, two weights' names and the row's size")
+        self.norm_weights: Optional[List[torch.Tensor]] = None
 
     def cache_spec(self):
         for m in self.members:
@@ -64,6 +74,7 @@ class SideBySide(Mixer):
         out = {}
         for m in self.members:
             out.update(m.param_specs())
+        out.update({name: ParamSpec((self.hidden_size,), role="vector", init="norm") for name in self.out_norms})
         return out
 
     def copies(self):
@@ -75,8 +86,16 @@ class SideBySide(Mixer):
     def load(self, get: TensorGetter) -> None:
         for m in self.members:
             m.load(get)
+        if self.out_norms:
+            self.norm_weights = [get(name, "vector").float().contiguous() for name in self.out_norms]
 
-    def forward(self, x, ctx, cache: LayerCache):
+    def forward_addends(self, x, ctx, cache: LayerCache) -> List[Addend]:
+        rows = self._results(x, ctx, cache)
+        if self.norm_weights is None:
+            return [Addend(r, factor=s) for r, s in zip(rows, self.scales)]
+        return [Addend(r, w, self.out_norm_eps, s) for r, w, s in zip(rows, self.norm_weights, self.scales)]
+
+    def _results(self, x, ctx, cache: LayerCache) -> List[torch.Tensor]:
         results = []
         for m, span in zip(self.members, self._state_at):
             state = cache.state[:, span[0]:span[1]] if span is not None and cache.state is not None else None
@@ -87,6 +106,15 @@ class SideBySide(Mixer):
             if bias is not None:
                 out = out + bias.float()
             results.append(out.contiguous())
+        return results
+
+    def forward(self, x, ctx, cache: LayerCache):
+        results = self._results(x, ctx, cache)
+        if self.norm_weights is not None:
+            total = torch.zeros_like(results[0])
+            for rows, weight, scale in zip(results, self.norm_weights, self.scales):
+                kernels.add_norm_mix(total, delta=rows, delta_weight=weight * scale, delta_eps=self.out_norm_eps)
+            return total, None
         total = torch.empty_like(results[0])
         kernels.scaled_sum(results[0], self.scales[0], results[1], self.scales[1], total)
         return total, None
