@@ -35,6 +35,9 @@ kept first tokens, latent attention with query latents, sinks, gates and shared 
 feed-forward behind norms and input filters of its own).
 ``--compare zasudra [--size 1k|2k]`` does the same for the Zasudra decoder (chunked attention, a wkv recurrence, gated
 attention that may read another layer's keys, routed squared-ReLU experts).
+``--compare zavizen [--size 1k|2k]`` does the same for the Zavizen decoder (hyper-connected streams, attention beside
+retention, a state-space mixer, routed experts in groups).
+
 ``--compare nufolix [--size 1k|2k]`` does the same for the Nufolix decoder (a state-space mixer; sigmoid attention with
 mixed heads side by side with a gated delta rule; dense xIELU feed-forwards).
 
@@ -982,13 +985,76 @@ def zasudra_work(z, tokens, keys_per_token, decode, requests=1):
     return work
 
 
+# ``--compare zavizen``: the same two measurements for the Zavizen decoder: four layers of hyper-connected streams (causal
+# attention with row norms beside retention, with a dense feed-forward; a state-space mixer with routed experts; attention
+# beside retention with routed experts; a state-space mixer with a dense feed-forward), beside a Qwen3 dense decoder of the
+# same width, depth and vocabulary whose attention has the same heads of 128.
+ZAVIZEN_SIZES = {
+    "1k": {"width": 1024, "streams": 4, "heads": 8, "kv_heads": 4, "dim": 128, "rot": 64, "ret_heads": 8, "ret_dim": 64, "ret_vdim": 128,
+           "ssm_heads": 16, "ssm_vdim": 128, "state": 64, "groups": 4, "conv": 4, "norm_groups": 4, "experts": 16, "top": 4,
+           "expert_ff": 1024, "shared_ff": 1024, "expert_groups": 4, "keep": 2, "ff": 4096, "layers": 4, "vocab": 32000, "qwen_heads": (8, 4)},
+    "2k": {"width": 2048, "streams": 4, "heads": 16, "kv_heads": 8, "dim": 128, "rot": 64, "ret_heads": 16, "ret_dim": 128, "ret_vdim": 128,
+           "ssm_heads": 32, "ssm_vdim": 128, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8, "experts": 32, "top": 4,
+           "expert_ff": 1408, "shared_ff": 2048, "expert_groups": 8, "keep": 4, "ff": 8192, "layers": 4, "vocab": 32000, "qwen_heads": (16, 8)},
+}
+
+
+def zavizen_config(z):
+    H = z["ret_heads"]
+    parallel = {"left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                         "rot": {"base": 500000.0, "dims": z["rot"], "scaling": {"factor": 2.0}}},
+                "right": {"heads": H, "dim": z["ret_dim"], "vdim": z["ret_vdim"], "rot": {"base": 10000.0, "dims": z["ret_dim"]},
+                          "decay": [1.0 - 2.0 ** -(5.0 + 5.0 * h / H) for h in range(H)]}}
+    ssm = {"heads": z["ssm_heads"], "vdim": z["ssm_vdim"], "state": z["state"], "groups": z["groups"], "conv": z["conv"],
+           "norm_groups": z["norm_groups"]}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "shared": {"ff": z["shared_ff"]},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5, "groups": {"count": z["expert_groups"], "keep": z["keep"]}}}
+    kinds = [("parallel", parallel, dense), ("mamba2", ssm, moe), ("parallel", parallel, moe), ("mamba2", ssm, dense)]
+    return {"architecture": "Zavizen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "streams": z["streams"],
+            "layers": [dict(zip(("type", "mixer", "mlp"), kinds[i % 4])) for i in range(z["layers"])]}
+
+
+def zavizen_work(z, tokens, keys_per_token, decode, requests=1):
+    """Closed-form work of the design's own kernel classes for one step: label -> (bytes, flops)."""
+    D, L, S = z["width"], z["layers"], z["streams"]
+    par, ssm, moe = (L + 1) // 2, L // 2, (L + 2) // 4 + (L + 1) // 4      # layers of each kind
+    H, G, d = z["heads"], z["kv_heads"], z["dim"]
+    Hr, dr, vr = z["ret_heads"], z["ret_dim"], z["ret_vdim"]
+    inner, channels = z["ssm_heads"] * z["ssm_vdim"], z["ssm_heads"] * z["ssm_vdim"] + 2 * z["groups"] * z["state"]
+    work = {}
+    # per sublayer: the streams read and written, the normed row written, one addend read (two where two mixers or an
+    # expert sum and a shared expert stand beside each other)
+    work["stream_step"] = (tokens * D * (2 * L * (8 * S + 2) + 4 * (2 * L + par + moe)), 0.0)
+    work["capped_rows_post"] = (par * tokens * (H + 2 * G) * d * (4 + 2), 0.0)
+    work["short_conv"] = (ssm * tokens * channels * 8, 0.0)
+    # queries, keys and values in, read-outs out, every request's state read and written once
+    work["retention_scan"] = (par * (tokens * Hr * 4 * (2 * dr + 2 * vr) + requests * Hr * dr * vr * 8), 0.0)
+    work["ssd_scan"] = (ssm * (tokens * 4 * (channels + inner) + requests * z["ssm_heads"] * z["state"] * z["ssm_vdim"] * 8), 0.0)
+    work["rotate_heads"] = (par * tokens * 2 * Hr * dr * 8, 0.0)
+    work["gated_group_norm"] = (tokens * (ssm * inner + par * Hr * vr) * (4 + 4 + 2), 0.0)
+    work["swiglu"] = (tokens * 6 * ((L - moe) * z["ff"] + moe * z["shared_ff"]), 0.0)
+    if decode:
+        work["capped_attention_mma"] = (par * tokens * 2 * 2 * keys_per_token * G * d, 0.0)
+    else:
+        work["capped_attention_mma"] = (0.0, par * 4.0 * tokens * keys_per_token * H * d)
+    pairs = tokens * z["top"]
+    if decode:
+        work["expert_rows"] = (moe * pairs * 3 * z["expert_ff"] * D * 2, 0.0)
+    else:
+        work["expert_rows"] = (0.0, moe * 2.0 * pairs * 3 * z["expert_ff"] * D)
+    work["expert_grouped"] = work["expert_tc"] = work["expert_rows"]
+    return work
+
+
 def run_compare(args):
     peak = peaks()
     sizes, config_of, work_of = {"zupilorn": (ZUPILORN_SIZES, zupilorn_config, zupilorn_work),
                                  "razelorn": (RAZELORN_SIZES, razelorn_config, razelorn_work),
                                  "nufolix": (NUFOLIX_SIZES, nufolix_config, lambda z, n, k, d: nufolix_work(z, n, k, d, args.batch if d else 1)),
                                  "tupidra": (TUPIDRA_SIZES, tupidra_config, lambda z, n, k, d: tupidra_work(z, n, k, d, args.batch if d else 1)),
-                                 "zasudra": (ZASUDRA_SIZES, zasudra_config, lambda z, n, k, d: zasudra_work(z, n, k, d, args.batch if d else 1))}[args.compare]
+                                 "zasudra": (ZASUDRA_SIZES, zasudra_config, lambda z, n, k, d: zasudra_work(z, n, k, d, args.batch if d else 1)),
+                                 "zavizen": (ZAVIZEN_SIZES, zavizen_config, lambda z, n, k, d: zavizen_work(z, n, k, d, args.batch if d else 1))}[args.compare]
     z = sizes[args.size]
     clocks = ClockSampler()
     clocks.start()
@@ -1084,7 +1150,7 @@ def main() -> int:
     parser.add_argument("--lean", action="store_true", help="leave out the per-kernel breakdown, the page-size point, the plain "
                         "PyTorch baseline and the self-check")
     parser.add_argument("--page-size", type=int, default=PAGE_SIZE, help="tokens per page of the key/value cache")
-    parser.add_argument("--compare", default="", choices=("", "zupilorn", "razelorn", "nufolix", "tupidra", "zasudra"),
+    parser.add_argument("--compare", default="", choices=("", "zupilorn", "razelorn", "nufolix", "tupidra", "zasudra", "zavizen"),
                         help="instead of the headline: prefill and decode of this design at real layer sizes beside a Qwen3 dense "
                         "decoder of the same width and depth, with the time of every kernel class")
     parser.add_argument("--size", default="2k", choices=tuple(ZUPILORN_SIZES), help="with --compare: the layer sizes")
