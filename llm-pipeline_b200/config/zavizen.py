@@ -166,7 +166,7 @@ class ZavizenConfig(ModelConfig):
                             out.append(f"router.groups must cut the experts into equal groups and keep some of them, got {groups}")
                         elif keep * (int(router["experts"]) // count) < int(router["top"]):
                             out.append(f"{keep} groups of {int(router['experts']) // count} experts do not hold {router['top']}")
-                if shared and shared.get("ff") is None:
+                if shared is not None and shared.get("ff") is None:
                     out.append("a shared expert needs shared.ff")
         return out
 
@@ -185,6 +185,8 @@ class ZavizenConfig(ModelConfig):
 
         total = 0
         for spec in expected_params(self.model_spec()).values():
+            if spec.optional:
+                continue
             count = 1
             for n in spec.shape:
                 count *= n if n is not None else 0

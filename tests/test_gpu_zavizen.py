@@ -1,0 +1,433 @@
+"""The Zavizen decoder in the engine against the plain implementation (``plain_zavizen.py``, float64): each mechanism alone,
+whole prompts, token-by-token decoding, portions down to two tokens, unequal batches, pages and slots used again, keys far
+away and at page borders, states carried over hundreds of tokens, looped layers, several shapes, long decoding through
+replayed graphs, and greedy generation through the entry point."""
+
+import itertools
+import math
+
+import pytest
+import torch
+
+import helpers as H
+import plain_zavizen as plain
+import zavizen_cases as Z
+
+pytestmark = pytest.mark.gpu
+DTYPES = [pytest.param(torch.float32, id="f32"), pytest.param(torch.bfloat16, id="bf16")]
+DEV = "cuda"
+
+
+def case(tmp_path, name, seed, sharp=None, slow=False, decided=False):
+    cfg = Z.CONFIGS[name] if sharp is None else Z.sharpen(Z.CONFIGS[name], sharp)
+    if decided:
+        cfg = Z.decided(cfg)
+    W = Z.weights_for(cfg, seed, slow=slow)
+    return cfg, W, Z.write_model(str(tmp_path), cfg, W)
+
+
+def requests_for(cfg, lengths, seed):
+    return {f"r{i}": H.random_tokens(cfg["vocab"], n, seed + i) for i, n in enumerate(lengths)}
+
+
+def _i32(values):
+    return torch.tensor(values, dtype=torch.int32, device=DEV)
+
+
+def _rel(got, want):
+    return float((got.double().cpu() - want).abs().max() / want.abs().max())
+
+
+def _portions(sizes_of_steps):
+    """For steps given as {slot: tokens}: (positions, q_start, slots) per step, and the (slot, first, end) of every request's rows."""
+    done = {}
+    for sizes in sizes_of_steps:
+        spans = []
+        for s, n in sizes.items():
+            spans.append((s, done.get(s, 0), done.get(s, 0) + n))
+            done[s] = done.get(s, 0) + n
+        yield (_i32([p for _s, a, b in spans for p in range(a, b)]), _i32([0] + list(itertools.accumulate(b - a for _s, a, b in spans))),
+               _i32(list(sizes)), spans)
+
+
+# ---- kernels alone ---------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("streams, width", [(1, 64), (2, 54), (3, 256), (4, 2052), (4, 5000), (5, 96), (6, 2400), (7, 40), (8, 4096), (16, 72)])
+def test_hyper_connections_alone(dtype, streams, width):
+    """Every form of the kernel: streams that are still one row, the first update and later ones in place, one addend and two,
+    with and without norms and scale, the combined row normed and plain, chosen rows that leave the streams alone."""
+    from llm_pipeline_b200.ops import kernels
+    gen = torch.Generator().manual_seed(streams * width)
+    T, eps = 9, 1e-5
+    rnd = lambda *s: torch.randn(*s, generator=gen)                                     # noqa: E731
+    xs, y0, y1 = rnd(T, streams, width), rnd(T, width) * 5.0, rnd(T, width) * 0.1
+    w0, w1, scale, nw = (rnd(width) * 0.3 + 1.0 for _ in range(4))
+    mix, into, out_w = rnd(streams, streams), rnd(streams), rnd(streams)
+    tol = 3e-6 if dtype == torch.float32 else 1e-2
+    dev = lambda t: t.to(DEV)                                                           # noqa: E731
+    D = lambda t: t.double()                                                            # noqa: E731
+    for first in (True, False):
+        x = xs[:, :1].expand(-1, streams, -1).contiguous() if first else xs
+        src = dev(xs[:, 0].contiguous()) if first else dev(x)
+        for addends, scaled in (((0,), False), ((0,), True), ((0, 1), True), ((1, 0), False)):
+            for normed in ((False, False), (True, True), (False, True), (True, False)):
+                ys = [(y0, y1)[j].to(dtype) for j in addends]
+                ws = [(w0, w1)[j] if normed[j] else None for j in addends]
+                y = sum((0.5 + j) * (plain.rms(D(t), eps, D(w)) if w is not None else D(t)) for j, (t, w) in enumerate(zip(ys, ws)))
+                y = y * D(scale) if scaled else y
+                want = torch.einsum("st,nsd->ntd", D(mix), D(x)) + D(out_w)[None, :, None] * y[:, None, :]
+                seen = torch.einsum("s,nsd->nd", D(into), want)
+                dst = torch.empty(T, streams, width, device=DEV) if first else src.clone()
+                out = torch.empty(T, width, device=DEV, dtype=dtype)
+                kernels.stream_step(src if first else dst, streams, dst=dst, addends=[(dev(t), dev(w) if w is not None else None, eps, 0.5 + j)
+                                                                                      for j, (t, w) in enumerate(zip(ys, ws))],
+                                    scale=dev(scale) if scaled else None, mix=dev(mix), out_weights=dev(out_w), in_weights=dev(into),
+                                    weight=dev(nw), eps=eps, out=out)
+                assert _rel(dst, want) < 3e-6 and _rel(out, plain.rms(seen, eps, D(nw))) < tol, (first, addends, normed)
+        # chosen rows: the plain sum normed, the streams as they were; and reading without an update
+        before, rows = src.clone(), _i32([7, 0, 3])
+        out = torch.empty(3, width, device=DEV, dtype=dtype)
+        kernels.stream_step(src, streams, addends=[(dev(y0), None, 0.0, 1.0)], mix=dev(mix), out_weights=dev(out_w), weight=dev(nw), eps=eps,
+                            out=out, rows=rows)
+        want = (torch.einsum("st,nsd->ntd", D(mix), D(x)) + D(out_w)[None, :, None] * D(y0)[:, None, :]).sum(dim=1)
+        assert _rel(out, plain.rms(want, eps, D(nw))[[7, 0, 3]]) < tol and torch.equal(src, before)
+        out = torch.empty(T, width, device=DEV)
+        kernels.stream_step(src, streams, in_weights=dev(into), out=out)
+        assert _rel(out, torch.einsum("s,nsd->nd", D(into), D(x))) < 3e-6
+
+
+@pytest.mark.parametrize("heads, dim, rot, shift", [(3, 16, 8, 0), (2, 33, 6, 1), (4, 7, 0, 0), (1, 128, 128, 0), (5, 64, 62, 4)])
+def test_rotation_of_query_and_key_heads_alone(heads, dim, rot, shift):
+    from llm_pipeline_b200.ops import kernels
+    gen = torch.Generator().manual_seed(dim)
+    n, base, factor = 21, 40.0, 3.0
+    rule = {"base": base, "dims": rot, "scaling": {"factor": factor}}
+    wide = torch.randn(n, 2 * heads * dim + shift, generator=gen)
+    x = wide[:, shift:].double().view(n, 2 * heads, dim)
+    want = plain.rotate(x, rule)
+    want[:, heads:] *= dim ** -0.5
+    cos = sin = None
+    if rot:
+        inv = torch.tensor([base ** (-2.0 * i / rot) / factor for i in range(rot // 2)], device=DEV)
+        cos, sin = torch.empty(n, rot // 2, device=DEV), torch.empty(n, rot // 2, device=DEV)
+        kernels.rope_tables(torch.arange(n, dtype=torch.int32, device=DEV), inv, 1.0, cos, sin)
+    got = wide.to(DEV)
+    kernels.rotate_heads(got[:, shift:], cos, sin, rot, 2 * heads, heads, dim, dim ** -0.5)
+    assert _rel(got[:, shift:], want.reshape(n, -1)) < 2e-6 and torch.equal(got[:, :shift].cpu(), wide[:, :shift])
+
+
+RETENTION_SIZES = [(3, 16, 20), (2, 20, 7), (1, 5, 64), (2, 64, 64), (1, 100, 33), (2, 128, 128), (4, 32, 48), (5, 1, 3), (1, 256, 512)]
+
+
+@pytest.mark.parametrize("sizes", RETENTION_SIZES, ids=str)
+def test_the_retention_recurrence_alone(sizes):
+    """On given rows, whole and cut into portions down to one token, in a slot that is not the first; decays of zero, of one and
+    between; the state of other slots and the entries around the piece stay as they are."""
+    from llm_pipeline_b200.ops import kernels
+    heads, dim, vdim = sizes
+    gen = torch.Generator().manual_seed(heads * dim)
+    n, Q, V = 75, heads * dim, heads * vdim
+    decay = ([0.997, 0.0, 1.0, 0.8, 0.95] * 2)[:heads]
+    rows = torch.randn(n, 2 * Q + V + 3, generator=gen)
+    q, k, v = rows[:, :Q], rows[:, Q:2 * Q], rows[:, 2 * Q:2 * Q + V]
+    want, _ = plain.retention_scan(q.double().view(n, heads, dim), k.double().view(n, heads, dim), v.double().view(n, heads, vdim),
+                                   torch.tensor(decay, dtype=torch.float64))
+    want = want.reshape(n, V)
+    exact = torch.tensor(decay, dtype=torch.float64)
+    decays = torch.stack([exact.float(), (exact - exact.float().double()).float()]).to(DEV)
+    rd = rows.to(DEV)
+    for cuts in ((), (1,), (1, 2, 4, 9, 10, 41), tuple(range(1, n)), (5, 50)):
+        out = torch.full((n, V), float("nan"), device=DEV)
+        offset, entries = 6, 2 * heads * dim * vdim
+        state = torch.full((4, offset + entries + 3), 5.0, device=DEV)
+        state[2] = 0.0
+        edges = [0] + list(cuts) + [n]
+        for lo, hi in zip(edges[:-1], edges[1:]):
+            part = rd[lo:hi]
+            kernels.retention_scan(part[:, :Q], part[:, Q:2 * Q], part[:, 2 * Q:2 * Q + V], decays, state, offset, _i32([0, hi - lo]), _i32([2]),
+                                   _i32(list(range(lo, hi))), out[lo:hi], heads, dim, vdim)
+        assert _rel(out, want) < 5e-6, cuts
+        assert (state[[0, 1, 3]] == 5.0).all() and (state[2, :offset] == 0.0).all() and (state[2, offset + entries:] == 0.0).all()
+
+
+def test_the_retention_recurrence_of_several_requests_at_once():
+    """Requests of unequal length in one step, from the states earlier steps left."""
+    from llm_pipeline_b200.ops import kernels
+    heads, dim, vdim = 2, 24, 40
+    Q, V = heads * dim, heads * vdim
+    gen = torch.Generator().manual_seed(3)
+    decay = torch.tensor([0.99, 0.6], dtype=torch.float64)
+    decays = torch.stack([decay.float(), (decay - decay.float().double()).float()]).to(DEV)
+    rows = {s: torch.randn(n, 2 * Q + V, generator=gen) for s, n in ((4, 60), (0, 1 + 33), (2, 2 + 8))}
+    want = {s: plain.retention_scan(x[:, :Q].double().view(-1, heads, dim), x[:, Q:2 * Q].double().view(-1, heads, dim),
+                                    x[:, 2 * Q:].double().view(-1, heads, vdim), decay)[0].reshape(-1, V) for s, x in rows.items()}
+    state = torch.zeros(5, 2 * heads * dim * vdim, device=DEV)
+    for positions, q_start, slots, spans in _portions([{4: 7}, {0: 1, 2: 2}, {4: 53, 0: 33, 2: 8}]):
+        x = torch.cat([rows[s][a:b] for s, a, b in spans]).to(DEV)
+        out = torch.empty(x.shape[0], V, device=DEV)
+        kernels.retention_scan(x[:, :Q], x[:, Q:2 * Q], x[:, 2 * Q:], decays, state, 0, q_start, slots, positions, out, heads, dim, vdim)
+        assert _rel(out, torch.cat([want[s][a:b] for s, a, b in spans])) < 5e-6
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads, dim", [(3, 16), (2, 20), (1, 100), (3, 7), (2, 600)])
+def test_heads_norm_and_silu_gate_alone(dtype, heads, dim):
+    from llm_pipeline_b200.ops import kernels
+    gen = torch.Generator().manual_seed(dim)
+    n, C, eps = 9, heads * dim, 1e-5
+    o, z = torch.randn(n, C, generator=gen) * 30.0, torch.randn(n, C, generator=gen) * 2.0
+    want = plain.rms(o.double().view(n, heads, dim), eps).reshape(n, C) * plain.silu(z.double())
+    out = kernels.gated_group_norm(o.to(DEV), z.to(DEV), None, torch.empty(n, C, device=DEV, dtype=dtype), dim, eps, gate_first=False)
+    assert _rel(out, want) < (3e-6 if dtype == torch.float32 else 1e-2)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("tokens, width, experts, top, groups, factor", [(3, 64, 6, 2, (3, 1), 1.0), (70, 54, 9, 4, (3, 2), 2.5), (200, 256, 64, 8, (8, 3), 0.7),
+                                                                     (65, 40, 3, 3, None, 1.3), (130, 48, 40, 1, (40, 1), 2.0), (20, 72, 16, 5, (2, 2), 1.0)])
+def test_router_with_groups_normalised_and_scaled_weights(dtype, tokens, width, experts, top, groups, factor):
+    from llm_pipeline_b200.ops import kernels
+    gen = torch.Generator().manual_seed(experts)
+    h, wr = torch.randn(tokens, width, generator=gen).to(dtype), torch.randn(experts, width, generator=gen) * 2.0 / math.sqrt(width)
+    ids = torch.full((tokens, top), -1, dtype=torch.int32, device=DEV)
+    weights = torch.full((tokens, top), float("nan"), device=DEV)
+    count, keep = groups or (0, 0)
+    kernels.route_topk(h.to(DEV), wr.to(DEV), top, ids, weights, score="softmax", groups=count, keep=keep, normalize=True, factor=factor)
+    rule = {"experts": experts, "top": top, "scale": factor, **({"groups": {"count": count, "keep": keep}} if groups else {})}
+    chosen, want = plain.route(h.double(), wr.double(), rule)
+    z = torch.sort(torch.log_softmax(h.double() @ wr.double().T, dim=-1), dim=-1, descending=True).values
+    clear = (z.diff(dim=1).abs() > 1e-5).all(dim=1)                            # no close call anywhere
+    assert clear.float().mean() > 0.8
+    assert torch.equal(ids.cpu().long()[clear], chosen[clear]) and _rel(weights.cpu()[clear], want[clear]) < 2e-5
+    assert (weights.sum(dim=1) - factor).abs().max() < 1e-5 * factor
+    if groups and keep < count:                                                # the premise: the limit changes choices
+        free, _ = plain.route(h.double(), wr.double(), {"experts": experts, "top": top})
+        assert experts // count == 1 or (free.sort(dim=1).values != chosen.sort(dim=1).values).any()
+
+
+# ---- one layer of each kind ------------------------------------------------------------------------------------------
+ONE_LAYER = {
+    "parallel": Z.config([Z.parallel((4, 2, 16, 24), (2, 12, 16), Z.dense(40), Z.rot(8), Z.rot(12))], width=40, vocab=50),
+    "parallel, bare": Z.config([Z.parallel((3, 1, 12, 10), (3, 7, 5))], streams=1, width=24, vocab=50),
+    "parallel, experts": Z.config([Z.parallel((2, 2, 16, 16), (1, 16, 40), Z.moe(24, 6, 2, (2, 1), 16), Z.rot(16, 30.0, 2.0), None, [0.9])], width=32, vocab=50),
+    "state space": Z.config([Z.mamba2(4, 12, 16, 2, 4, 2, Z.moe(24, 4, 1))], streams=4, width=40, vocab=50),
+    "state space, bare": Z.config([Z.mamba2(3, 5, 7, 1, 2, 1)], streams=3, width=30, vocab=50),
+    "one layer looped": Z.config([Z.parallel((2, 1, 16, 16), (2, 8, 8), Z.dense(24), Z.rot(4), Z.rot(8))], streams=2, width=32, vocab=50, loop=(0, 1, 4)),
+}
+
+
+@pytest.mark.parametrize("name", sorted(ONE_LAYER))
+def test_one_layer_alone(tmp_path, name):
+    cfg = ONE_LAYER[name]
+    W = Z.weights_for(cfg, 11)
+    folder = Z.write_model(str(tmp_path), cfg, W)
+    requests = requests_for(cfg, [1, 2, 33, 70], 50)
+    want = Z.oracle(cfg, W, requests)
+    runner = H.make_runner(folder, torch.float32, page_size=8, num_pages=24, max_request_tokens=96, max_requests=2)
+    Z.assert_matches(H.replay(runner, H.cut_whole(requests)), want, torch.float32, f"{name}, whole")
+    Z.assert_matches(H.replay(runner, H.cut_portions(requests, (2, 5, 1, 16))), want, torch.float32, f"{name}, portions")
+
+
+def test_the_sum_of_streams_after_every_layer_run(tmp_path):
+    """float32, layer run by layer run (looped layers once per pass): the streams' sum against the plain implementation's."""
+    from llm_pipeline_b200.engine import StepEntry
+    for name in ("mixed", "all_looped"):
+        cfg, W, folder = case(tmp_path / name, name, 13)
+        tokens = H.random_tokens(cfg["vocab"], 40, 5)
+        want = []
+        plain.forward(cfg, W, tokens, want)
+        runner = H.make_runner(folder, torch.float32, page_size=8, num_pages=8, max_request_tokens=64, max_requests=1)
+        ctx = runner._prepare([StepEntry("a", tokens, [0])])
+        stream = runner.model.begin(ctx, runner._views)
+        for index, ref in enumerate(want):
+            runner.model.run_layers(ctx, runner._views, stream, index, index + 1)
+            assert _rel(stream.settle().sum(dim=1), ref) < 2e-5, (name, index)
+        assert len(want) == len(runner.model.schedule)
+
+
+# ---- whole models ----------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", sorted(Z.CONFIGS))
+def test_prefill_decoding_portions_and_batches(tmp_path, name, dtype):
+    cfg, W, folder = case(tmp_path, name, 3, decided=dtype == torch.bfloat16)
+    requests = requests_for(cfg, [1, 2, 3, 19, 64, 65, 150], 100)
+    want = Z.oracle(cfg, W, requests)
+    page = 8
+    share = 1.0 if dtype == torch.float32 else 0.97
+    runner = H.make_runner(folder, dtype, page_size=page, num_pages=2 * (-(-150 // page)) + 6, max_request_tokens=160, max_requests=4)
+    Z.assert_matches(H.replay(runner, H.cut_whole(requests)), want, dtype, f"{name}: whole prompts", share)
+    Z.assert_matches(H.replay(runner, H.cut_tail_one_by_one(requests, tail=40)), want, dtype, f"{name}: last tokens one by one", share)
+    Z.assert_matches(H.replay(runner, H.cut_portions(requests, (1,))), want, dtype, f"{name}: token by token", share)
+    Z.assert_matches(H.replay(runner, H.cut_portions(requests, (2, 7, 3, 64, 2, 33))), want, dtype, f"{name}: portions", share)
+    # unequal requests side by side, four live at most, so the slots and pages of finished ones go to later ones
+    got = H.replay(runner, H.cut_mixed(requests, (2, 5, 16, 3, 31), max_live=4, decode_tail=9))
+    Z.assert_matches(got, want, dtype, f"{name}: mixed batches", share)
+    assert runner.cache.num_live == 0 and runner.cache.pages_reused > 0         # seven requests went through four slots
+
+
+def test_routed_choices_in_bfloat16(tmp_path):
+    """With a router that chooses, bfloat16 may flip a close call, which then moves the rows after it: most rows still agree."""
+    cfg, W, folder = case(tmp_path, "one_stream", 23)
+    requests = requests_for(cfg, [40, 25, 9], 150)
+    want = Z.oracle(cfg, W, requests)
+    runner = H.make_runner(folder, torch.bfloat16, page_size=16, num_pages=12, max_request_tokens=48, max_requests=3)
+    Z.assert_matches(H.replay(runner, H.cut_whole(requests)), want, torch.bfloat16, "routed choices", 0.8)
+
+
+def test_the_same_logits_alone_and_in_a_batch(tmp_path):
+    """float32: a request's logits beside others, or cut into portions, are those it has alone, to rounding of sums."""
+    cfg, W, folder = case(tmp_path, "mixed", 4)
+    requests = requests_for(cfg, [5, 40, 77, 130], 200)
+    runner = H.make_runner(folder, torch.float32, page_size=16, num_pages=24, max_request_tokens=144, max_requests=4)
+    alone = H.replay(runner, H.cut_whole(requests))
+    mixed = H.replay(runner, H.cut_mixed(requests, (3, 2, 17), max_live=4, decode_tail=5))
+    for rid in requests:
+        assert (alone[rid] - mixed[rid]).abs().max() < 2e-4 * alone[rid].abs().max(), rid
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["mixed", "one_stream", "wide_heads"])
+def test_far_keys_and_page_borders_under_a_sharp_softmax(tmp_path, name, dtype):
+    """Scores of a wide spread: a query's weight sits on one or two keys, often hundreds of tokens back, so a key that is lost,
+    off by one or read from another request's page changes the logits by its whole value. Prompts as long as many pages,
+    positions around every page border, decoded alone and in portions."""
+    cfg, W, folder = case(tmp_path, name, 5, sharp=4.0, decided=dtype == torch.bfloat16)
+    page = 16
+    requests = requests_for(cfg, [4 * page, 4 * page + 1, 330, 17], 300)
+    want = Z.oracle(cfg, W, requests)
+    # the premise: in the plain implementation itself the far keys matter (without the first 3 pages the late logits differ much)
+    late = plain.forward(cfg, W, requests["r2"][3 * page:]).float()
+    assert Z.row_errors(late[-40:], want["r2"][-40:]).median() > 0.03
+    runner = H.make_runner(folder, dtype, page_size=page, num_pages=2 * 21 + 4, max_request_tokens=336, max_requests=4)
+    share = 1.0 if dtype == torch.float32 else 0.95
+    Z.assert_matches(H.replay(runner, H.cut_whole(requests)), want, dtype, "sharp: whole", share)
+    Z.assert_matches(H.replay(runner, H.cut_tail_one_by_one(requests, tail=3 * page + 2)), want, dtype, "sharp: decoding across borders", share)
+    Z.assert_matches(H.replay(runner, H.cut_portions(requests, (page - 1, 2, page + 1, 2 * page, 3))), want, dtype, "sharp: portions", share)
+    Z.assert_matches(H.replay(runner, H.cut_mixed(requests, (page, 2, page + 1), max_live=3, decode_tail=page + 3)), want, dtype, "sharp: mixed", share)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_states_carry_what_was_written_hundreds_of_tokens_back(tmp_path, dtype):
+    """Decays close to one in both recurrences: what the first tokens wrote still weighs in the logits 300 tokens later, so a state
+    that is lost, zeroed at a cut, shared between the passes of a loop or taken from another slot shows."""
+    cfg = Z.config([Z.parallel((2, 1, 16, 16), (3, 16, 16), Z.dense(40), None, Z.rot(8, 1000.0), [0.996, 0.998, 1.0]),
+                    Z.mamba2(3, 16, 24, 3, 3, 1, Z.moe(24, 4, 4, None, 16))], streams=2, width=40, vocab=80, loop=(0, 2, 2))
+    W = Z.weights_for(cfg, 12, slow=True)
+    for name in W:                                                      # the states speak, the attention does not
+        if name.endswith("left.out"):
+            W[name] = W[name] * 0.0
+    folder = Z.write_model(str(tmp_path), cfg, W)
+    requests = requests_for(cfg, [320, 301, 47], 900)
+    want = Z.oracle(cfg, W, requests)
+    other = list(requests["r0"])
+    other[:8] = H.random_tokens(cfg["vocab"], 8, 77)                    # the premise: the first tokens still matter at the end
+    assert Z.row_errors(plain.forward(cfg, W, other).float()[-20:], want["r0"][-20:]).median() > 0.01
+    runner = H.make_runner(folder, dtype, page_size=16, num_pages=50, max_request_tokens=336, max_requests=3)
+    share = 1.0 if dtype == torch.float32 else 0.97
+    Z.assert_matches(H.replay(runner, H.cut_whole(requests)), want, dtype, "long memory: whole", share)
+    Z.assert_matches(H.replay(runner, H.cut_portions(requests, (2, 63, 1, 130, 5))), want, dtype, "long memory: portions", share)
+    Z.assert_matches(H.replay(runner, H.cut_mixed(requests, (40, 2, 9), max_live=2, decode_tail=20)), want, dtype, "long memory: mixed", share)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_long_prompts_and_decoding_over_key_segments(tmp_path, dtype, monkeypatch):
+    """Prompts long enough for the grouped expert products and contexts long enough for the attention's key segments in
+    decoding, eager and replayed; sharp enough that a far key shows."""
+    from llm_pipeline_b200.ops import kernels
+    cfg = Z.sharpen(Z.config([Z.parallel((4, 2, 16, 16), (2, 32, 32), Z.moe(32, 6, 6, (3, 3), 24), Z.rot(8, 1000.0, 2.0), Z.rot(32, 1000.0)),
+                              Z.mamba2(2, 32, 32, 1, 4, 2, Z.dense(64))], streams=4, width=48, vocab=90), 2.5)
+    W = Z.weights_for(cfg, 31)
+    folder = Z.write_model(str(tmp_path), cfg, W)
+    requests = requests_for(cfg, [700, 640], 500)
+    want = Z.oracle(cfg, W, requests)
+    used = {"keys": 0}
+    attend = kernels.capped_attention_mma
+
+    def counted_attend(*args, **kwargs):
+        used["keys"] += kwargs.get("segments", 0) > 1
+        return attend(*args, **kwargs)
+
+    monkeypatch.setattr(kernels, "capped_attention_mma", counted_attend)
+    runner = H.make_runner(folder, dtype, page_size=16, num_pages=90, max_request_tokens=720, max_requests=2)
+    share = 1.0 if dtype == torch.float32 else 0.97
+    Z.assert_matches(H.replay(runner, H.cut_whole(requests)), want, dtype, "long: whole", share)
+    Z.assert_matches(H.replay(runner, H.cut_portions(requests, (513, 2, 61, 1))), want, dtype, "long: portions", share)
+    Z.assert_matches(H.replay(runner, H.cut_mixed(requests, (520, 33), max_live=2, decode_tail=30)), want, dtype, "long: side by side", share)
+    assert (used["keys"] > 0) == (dtype == torch.bfloat16) and runner.graph_replays > 0
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_long_decoding_through_replayed_graphs(tmp_path, dtype):
+    """Two requests decode side by side for 220 steps over many pages, the states taking turns between their two copies: from the
+    third step on a captured graph is replayed."""
+    cfg, W, folder = case(tmp_path, "mixed", 6, decided=dtype == torch.bfloat16)
+    requests = requests_for(cfg, [260, 231], 400)
+    want = Z.oracle(cfg, W, requests)
+    runner = H.make_runner(folder, dtype, page_size=16, num_pages=40, max_request_tokens=272, max_requests=2)
+    from llm_pipeline_b200.engine import StepEntry
+    rows = {rid: [] for rid in requests}
+    out = runner.step([StepEntry(rid, toks[:11], list(range(11))) for rid, toks in requests.items()])
+    for k, rid in enumerate(requests):
+        rows[rid].append(out[11 * k:11 * (k + 1)].float().cpu())
+    for t in range(11, 231):
+        out = runner.step([StepEntry(rid, [toks[t]], [0]) for rid, toks in requests.items()])
+        for k, rid in enumerate(requests):
+            rows[rid].append(out[k:k + 1].float().cpu())
+    assert runner.graph_replays > 200
+    share = 1.0 if dtype == torch.float32 else 0.97
+    for rid in requests:
+        Z.assert_matches({rid: torch.cat(rows[rid])}, {rid: want[rid][:231]}, dtype, f"long decoding of {rid}", share)
+
+
+def test_decoding_with_layers_that_run_between_graphs(tmp_path, monkeypatch):
+    """A part that cannot be captured splits a decode step into graphs and eager layers; what crosses is all streams."""
+    cfg, W, folder = case(tmp_path, "mixed", 9)
+    requests = requests_for(cfg, [40, 33], 450)
+    want = Z.oracle(cfg, W, requests)
+    from llm_pipeline_b200.parts.state_space import StateSpaceDuality
+    monkeypatch.setattr(StateSpaceDuality, "graph_safe", False)
+    runner = H.make_runner(folder, torch.float32, page_size=16, num_pages=8, max_request_tokens=48, max_requests=2)
+    assert len(runner._pieces) == 6
+    Z.assert_matches(H.replay(runner, H.cut_tail_one_by_one(requests, tail=30)), want, torch.float32, "pieces")
+    assert runner.graph_replays > 40
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_greedy_generation_through_the_entry_point(tmp_path, dtype):
+    from llm_pipeline_b200.inference import InferenceConfig, InferenceEngine
+    cfg, W, folder = case(tmp_path, "all_looped" if dtype == torch.float32 else "one_stream", 7, decided=dtype == torch.bfloat16)
+    engine = InferenceEngine(InferenceConfig(model_path=folder, dtype=dtype, block_size=8, num_blocks=64, max_sequence_length=128,
+                                             max_batch_size=4, max_num_batched_tokens=32))
+    prompts = [H.random_tokens(cfg["vocab"], n, 600 + n) for n in (1, 7, 30, 45, 12)]       # five requests for four slots
+    got = engine.generate(prompts, max_tokens=10, temperature=0.0)
+    checked = 0
+    for prompt, tokens in zip(prompts, got):
+        ids = list(prompt)
+        for token in tokens:
+            logits = plain.forward(cfg, W, ids)[-1]
+            top2 = torch.topk(logits, 2).values
+            if dtype == torch.bfloat16 and float(top2[0] - top2[1]) < 0.04 * float(logits.std()) * 4:
+                break                                                   # a near tie: the two sequences may part here
+            assert token == int(logits.argmax()), (len(prompt), len(ids) - len(prompt))
+            ids.append(token)
+            checked += 1
+    assert checked >= (50 if dtype == torch.float32 else 15)
+    assert engine.engine.cache.num_live == 0
+    info = engine.get_model_info()
+    assert info["vocab_size"] == cfg["vocab"] and info["num_layers"] == len(cfg["layers"]) and info["total_parameters"] > 0
+
+
+def test_generation_with_a_preempted_request(tmp_path):
+    """Too few pages for all requests: one is preempted and computed again, its states from nothing."""
+    from llm_pipeline_b200.inference import InferenceConfig, InferenceEngine
+    cfg, W, folder = case(tmp_path, "mixed", 8)
+    engine = InferenceEngine(InferenceConfig(model_path=folder, dtype=torch.float32, block_size=8, num_blocks=12, max_sequence_length=64,
+                                             max_batch_size=3, max_num_batched_tokens=32))
+    prompts = [H.random_tokens(cfg["vocab"], n, 700 + n) for n in (25, 27, 21)]
+    got = engine.generate(prompts, max_tokens=16, temperature=0.0)
+    for prompt, tokens in zip(prompts, got):
+        ids = list(prompt)
+        for token in tokens:
+            assert token == int(plain.forward(cfg, W, ids)[-1].argmax())
+            ids.append(token)
+        assert len(tokens) == 16
+    assert engine.engine.cache.num_live == 0
