@@ -29,6 +29,7 @@ struct ScanArgs {
     const int* q_start; const int* slots; const int* positions;
     float* y; long y_t;                      // [tokens, H P]
     int H, G, N, P;
+    int max_tokens;                          // requests that bring more are left to other kernels
 };
 
 constexpr int SS_THREADS = 128;   // threads of a block that hold the state; one more warp copies the inputs
@@ -73,7 +74,7 @@ __global__ void __launch_bounds__(SS_THREADS + 32 * SS_COPY_WARPS) ssd_scan_kern
     constexpr int ROW = 2 * NP + COLS + 4;              // B, C (padded), the block's columns of x, dt, decay
     const int r = blockIdx.x, h = blockIdx.y;
     const int begin = a.q_start[r], end = a.q_start[r + 1];
-    if (end <= begin) return;
+    if (end <= begin || end - begin > a.max_tokens) return;
     const int N = a.N, P = a.P;
     const bool loader = threadIdx.x >= SS_THREADS;
     const int copy_warp = ((int)threadIdx.x - SS_THREADS) >> 5;      // which of the copying warps (negative for the others)
@@ -252,23 +253,23 @@ static int launch_scan(const ScanArgs& a, int R, cudaStream_t stream) {
 LLMP_API int llmp_ssd_scan(const float* xbc, long xbc_t, const float* dt, long dt_t, const float* dt_bias, const float* a_log,
                            const float* d_skip, float* state, long state_slot, long state_half, const int* q_start,
                            const int* slots, const int* positions, float* y, long y_t, int R, int H, int G, int N, int P,
-                           cudaStream_t stream) {
+                           int max_tokens, cudaStream_t stream) {
     ScanArgs a = {};
     a.x = xbc; a.x_t = xbc_t; a.b = xbc + (size_t)H * P; a.c = a.b + (size_t)G * N; a.bc_t = xbc_t;
     a.dt = dt; a.dt_t = dt_t; a.dt_bias = dt_bias; a.a_log = a_log; a.d_skip = d_skip;
     a.state = state; a.state_slot = state_slot; a.state_half = state_half; a.q_start = q_start; a.slots = slots;
-    a.positions = positions; a.y = y; a.y_t = y_t; a.H = H; a.G = G; a.N = N; a.P = P;
+    a.positions = positions; a.y = y; a.y_t = y_t; a.H = H; a.G = G; a.N = N; a.P = P; a.max_tokens = max_tokens;
     return launch_scan(a, R, stream);
 }
 
 // q, k [tokens, H N] and v [tokens, H P] with one stride; decay [2][H].
 LLMP_API int llmp_retention_scan(const float* q, const float* k, const float* v, long qkv_t, const float* decay, float* state,
                                  long state_slot, long state_half, const int* q_start, const int* slots, const int* positions,
-                                 float* y, long y_t, int R, int H, int N, int P, cudaStream_t stream) {
+                                 float* y, long y_t, int R, int H, int N, int P, int max_tokens, cudaStream_t stream) {
     ScanArgs a = {};
     a.x = v; a.x_t = qkv_t; a.b = k; a.c = q; a.bc_t = qkv_t; a.decay = decay;
     a.state = state; a.state_slot = state_slot; a.state_half = state_half; a.q_start = q_start; a.slots = slots;
-    a.positions = positions; a.y = y; a.y_t = y_t; a.H = H; a.G = H; a.N = N; a.P = P;
+    a.positions = positions; a.y = y; a.y_t = y_t; a.H = H; a.G = H; a.N = N; a.P = P; a.max_tokens = max_tokens;
     return launch_scan(a, R, stream);
 }
 

@@ -91,9 +91,10 @@ _SIGNATURES = {
     "llmp_diff_attention_mma": [_P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F,
                                 _I, _I, _I, _P, _P, _P],
     "llmp_short_conv": [_P, _L, _P, _I, _P, _I, _P, _L, _L, _P, _P, _P, _P, _P, _L, _P, _I, _L, _L, _I, _I, _I, _I, _I, _I, _I, _P],
-    "llmp_ssd_scan": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P],
-    "llmp_retention_scan": [_P, _P, _P, _L, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P],
-    "llmp_rotate_heads": [_P, _L, _P, _P, _I, _I, _I, _I, _F, _I, _P],
+    "llmp_ssd_scan": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _P],
+    "llmp_retention_scan": [_P, _P, _P, _L, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P],
+    "llmp_rotate_heads": [_P, _L, _P, _L, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
+    "llmp_chunked_scan": [_P, _P, _P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _P, _I, _P, _P, _P, _L, _I, _I, _I, _I, _P],
     "llmp_stream_step": [_P, _L, _L, _P, _P, _I, _P, _F, _F, _P, _I, _P, _F, _F, _P, _P, _P, _P, _P, _I, _F, _P, _I, _P, _I, _I, _I, _P],
     "llmp_gated_group_norm": [_P, _L, _P, _L, _P, _P, _I, _L, _I, _I, _I, _I, _F, _P],
     "llmp_delta_prep": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _I, _I, _I, _I, _P],
@@ -1317,12 +1318,16 @@ def short_conv(x: torch.Tensor, taps: torch.Tensor, bias: Optional[torch.Tensor]
     return out if out is not None else out_typed
 
 
+_ALL_TOKENS = 2 ** 31 - 1
+
+
 def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, d_skip: torch.Tensor,
              state: torch.Tensor, state_offset: int, q_start: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor,
-             y: torch.Tensor, heads: int, groups: int, state_size: int, vdim: int) -> torch.Tensor:
+             y: torch.Tensor, heads: int, groups: int, state_size: int, vdim: int, max_tokens: Optional[int] = None) -> torch.Tensor:
     """The state-space recurrence with a scalar decay per head and token (csrc/state_space.cu): ``xbc`` float32 [tokens,
     heads vdim + 2 groups state] = x | B | C, ``dt`` float32 [tokens, heads] (a view), the three per-head vectors float32,
-    ``y`` float32 [tokens, heads vdim]. The state piece holds two copies of [heads, state, vdim]."""
+    ``y`` float32 [tokens, heads vdim]. The state piece holds two copies of [heads, state, vdim]. ``max_tokens``: requests that
+    bring more are left alone (``chunked_scan`` takes them)."""
     N = xbc.shape[0]
     _need(xbc.dtype == torch.float32 and xbc.stride(1) == 1 and xbc.shape[1] == heads * vdim + 2 * groups * state_size,
           "ssd_scan: x | B | C has the wrong width")
@@ -1335,13 +1340,13 @@ def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: 
     ptr, slot_stride, half = _state_views(state, state_offset, heads * state_size * vdim, "ssd_scan")
     _call("llmp_ssd_scan", _ptr(xbc), xbc.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), ptr,
           slot_stride, half, _ptr(q_start), _ptr(slots), _ptr(positions), _ptr(y), y.stride(0), slots.numel(), heads, groups,
-          state_size, vdim, _stream())
+          state_size, vdim, _ALL_TOKENS if max_tokens is None else int(max_tokens), _stream())
     return y
 
 
 def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, state_offset: int,
                    q_start: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor, y: torch.Tensor, heads: int, dim: int,
-                   vdim: int) -> torch.Tensor:
+                   vdim: int, max_tokens: Optional[int] = None) -> torch.Tensor:
     """S <- decay[h] S + k_t v_t^T, y_t = S^T q_t per head (csrc/state_space.cu): ``q``, ``k`` float32 [tokens, heads dim] and ``v``
     [tokens, heads vdim], views with one stride between tokens; ``decay`` float32 [2, heads], the constants and what their
     float leaves of them; ``y`` float32 [tokens, heads vdim]. The state piece holds two copies of [heads, dim, vdim]."""
@@ -1354,20 +1359,75 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
         _i32(t, name)
     ptr, slot_stride, half = _state_views(state, state_offset, heads * dim * vdim, "retention_scan")
     _call("llmp_retention_scan", _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), ptr, slot_stride, half, _ptr(q_start), _ptr(slots),
-          _ptr(positions), _ptr(y), y.stride(0), slots.numel(), heads, dim, vdim, _stream())
+          _ptr(positions), _ptr(y), y.stride(0), slots.numel(), heads, dim, vdim, _ALL_TOKENS if max_tokens is None else int(max_tokens), _stream())
+    return y
+
+
+CHUNKED_SCAN_TOKENS = 128            # csrc/chunked_scan.cu: tokens of a chunk
+CHUNKED_SCAN_MIN_TOKENS = 32         # a request's tokens in a step from which its recurrences run in chunks
+
+
+def chunked_scan_supports(dtype: torch.dtype, state_size: int, vdim: int, state_offset: int, state_entries: int) -> bool:
+    """bfloat16, and a state whose rows and columns come in sixteens at a 16-byte boundary of the slot."""
+    return (dtype == torch.bfloat16 and state_size % 16 == 0 and 16 <= state_size <= 256 and vdim % 16 == 0 and vdim >= 16 and
+            state_offset % 4 == 0 and state_entries % 4 == 0)
+
+
+def plan_chunks(q_lens: Sequence[int], min_tokens: int):
+    """((first row, tokens) per chunk, (request, its first chunk, its chunks) per request of at least ``min_tokens``)."""
+    chunks, requests, row = [], [], 0
+    for r, n in enumerate(q_lens):
+        if n >= min_tokens:
+            first = len(chunks)
+            chunks += [(row + t, min(CHUNKED_SCAN_TOKENS, n - t)) for t in range(0, n, CHUNKED_SCAN_TOKENS)]
+            requests.append((r, first, len(chunks) - first))
+        row += n
+    return chunks, requests
+
+
+def chunked_scan(b: torch.Tensor, c: torch.Tensor, x: torch.Tensor, state: torch.Tensor, state_offset: int, q_start: torch.Tensor,
+                 slots: torch.Tensor, positions: torch.Tensor, chunks: torch.Tensor, requests: torch.Tensor, y: torch.Tensor, heads: int,
+                 groups: int, state_size: int, vdim: int, *, log_decay: Optional[torch.Tensor] = None, dt: Optional[torch.Tensor] = None,
+                 dt_bias: Optional[torch.Tensor] = None, a_log: Optional[torch.Tensor] = None, d_skip: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The recurrences of ``ssd_scan`` (with ``dt``, ``dt_bias``, ``a_log``, ``d_skip``) and ``retention_scan`` (with ``log_decay``
+    float32 [heads]; b, c, x are keys, queries, values) for requests of many tokens, in chunks on the tensor cores
+    (csrc/chunked_scan.cu). ``b``, ``c`` [tokens, groups state], ``x`` [tokens, heads vdim]: bfloat16 views with one stride between
+    tokens. ``chunks`` int32 [n, 2] and ``requests`` int32 [m, 3]: ``plan_chunks`` on the device. Rows of other requests, of
+    ``y`` too, are left alone."""
+    N = b.shape[0]
+    H, S, P = int(heads), int(state_size), int(vdim)
+    _need(all(t.dtype == torch.bfloat16 and t.stride(1) == 1 and t.stride(0) == b.stride(0) for t in (b, c, x)), "chunked_scan takes bfloat16 rows")
+    _need(b.shape == c.shape == (N, groups * S) and x.shape == (N, H * P), "chunked_scan: rows have the wrong shape")
+    _need(y.dtype == torch.float32 and y.stride(1) == 1 and y.shape == (N, H * P), "chunked_scan: y has the wrong shape")
+    _need((log_decay is None) == (dt is not None), "chunked_scan: constant decays, or step sizes")
+    for t in (log_decay,) if dt is None else (dt_bias, a_log, d_skip):
+        _need(t.dtype == torch.float32 and t.numel() == H and t.is_contiguous(), "chunked_scan takes float32 vectors of one entry per head")
+    _need(dt is None or (dt.dtype == torch.float32 and dt.stride(1) == 1 and dt.shape == (N, H)), "chunked_scan: dt must be float32 [tokens, heads]")
+    for t, name in ((q_start, "q_start"), (slots, "slots"), (positions, "positions"), (chunks, "chunks"), (requests, "requests")):
+        _i32(t, name)
+    n = chunks.shape[0]
+    sums = torch.empty((n, H, S, P), dtype=torch.float32, device=b.device)
+    gains = torch.empty((n, H), dtype=torch.float32, device=b.device)
+    ptr, slot_stride, half = _state_views(state, state_offset, H * S * P, "chunked_scan")
+    _call("llmp_chunked_scan", _ptr(b), _ptr(c), _ptr(x), b.stride(0), _ptr(dt), dt.stride(0) if dt is not None else 0, _ptr(dt_bias), _ptr(a_log),
+          _ptr(d_skip), _ptr(log_decay), ptr, slot_stride, half, _ptr(q_start), _ptr(slots), _ptr(positions), _ptr(chunks), n, _ptr(requests),
+          requests.shape[0], _ptr(sums), _ptr(gains), _ptr(y), y.stride(0), H, int(groups), S, P, _stream())
     return y
 
 
 def rotate_heads(x: torch.Tensor, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot: int, heads: int, scaled_from: int,
-                 dim: int, factor: float) -> torch.Tensor:
-    """In place on float32 rows of ``heads`` heads: entry i of the first ``rot`` of every head turns with entry i + rot / 2, and
-    the heads from ``scaled_from`` on are multiplied by ``factor`` afterwards."""
+                 dim: int, factor: float, typed: Optional[torch.Tensor] = None, in_place: bool = True) -> torch.Tensor:
+    """On float32 rows of ``heads`` heads: entry i of the first ``rot`` of every head turns with entry i + rot / 2, and the heads
+    from ``scaled_from`` on are multiplied by ``factor`` afterwards; ``in_place``, and / or into ``typed`` (bfloat16 rows), which
+    may have further columns: those of ``x`` behind the heads, as they are."""
     N = x.shape[0]
-    _need(x.dtype == torch.float32 and x.stride(1) == 1 and x.shape == (N, heads * dim), "rotate_heads takes float32 rows")
+    extra = typed.shape[1] - heads * dim if typed is not None else 0
+    _need(x.dtype == torch.float32 and x.stride(1) == 1 and extra >= 0 and x.shape == (N, heads * dim + extra), "rotate_heads takes float32 rows")
+    _need(typed is None or (typed.dtype == torch.bfloat16 and typed.stride(1) == 1 and typed.shape[0] == N), "rotate_heads gives bfloat16 rows")
     _need(rot == 0 or (cos.dtype == sin.dtype == torch.float32 and cos.is_contiguous() and sin.is_contiguous() and
                        cos.shape == sin.shape == (N, rot // 2)), "rotate_heads: rotary tables have the wrong shape")
-    _call("llmp_rotate_heads", _ptr(x), x.stride(0), _ptr(cos), _ptr(sin), int(rot), int(heads), int(scaled_from), int(dim), float(factor), N,
-          _stream())
+    _call("llmp_rotate_heads", _ptr(x), x.stride(0), _ptr(typed), typed.stride(0) if typed is not None else 0, 1 if in_place else 0, _ptr(cos),
+          _ptr(sin), int(rot), int(heads), int(scaled_from), int(dim), int(extra), float(factor), N, _stream())
     return x
 
 

@@ -9,7 +9,8 @@ With h the mixer's input, H heads with queries and keys of ``dim`` entries and v
 
 There is no softmax and no denominator. The four products that read h are one product against [Wq; Wk; Wv; Wg] with a float32
 result; rotation, decay, state, read-out, norm and gate are float32 (``csrc/retention.cu``, ``csrc/state_space.cu``: the
-recurrence is the state-space one with a constant decay, a step size of one and a group per head); the gated rows are rounded
+recurrence is the state-space one with a constant decay, a step size of one and a group per head); in bfloat16, requests of many
+tokens run in chunks on the tensor cores with the rotated q, k and the v rounded to bfloat16 (``csrc/chunked_scan.cu``); the gated rows are rounded
 once to the compute type for the output product, whose result is float32 again.
 
 State of a request: one float32 vector with two copies of [H, dim, vdim] that take turns by the parity of the last position
@@ -27,6 +28,7 @@ from ..ops.linear import linear
 from ..weights.source import ParamSpec
 from .base import LayerCache, Mixer, TensorGetter
 from .registry import register_mixer
+from .state_space import chunk_plan
 
 
 @register_mixer("retention")
@@ -49,7 +51,7 @@ class Retention(Mixer):
         self.qk_size, self.v_size = self.heads * self.dim, self.heads * self.vdim
         self.names = {n: n for n in ("q", "k", "v", "g", "o")}
         self.names.update(names or {})
-        self.w_in = self.w_out = self.decays = None
+        self.w_in = self.w_out = self.decays = self.log_decay = None
 
     def state_entries(self) -> int:
         return 2 * self.heads * self.dim * self.vdim
@@ -75,6 +77,8 @@ class Retention(Mixer):
         exact = torch.tensor(self.decay, dtype=torch.float64)
         high = exact.float()
         self.decays = torch.stack([high, (exact - high.double()).float()]).contiguous().to(self.w_out.device)
+        # a decay of zero: finite, and so far down that a token later nothing is left
+        self.log_decay = torch.log(exact).clamp(min=-1e30).float().to(self.w_out.device)
 
     def forward(self, x, ctx, cache: LayerCache):
         if cache.state is None:
@@ -82,10 +86,21 @@ class Retention(Mixer):
         N, Q, V = ctx.num_tokens, self.qk_size, self.v_size
         proj = linear(x, self.w_in, out_dtype=torch.float32)                # [N, q | k | v | gate]
         cos, sin = ctx.position_tables[self.position] if self.rotary_dim else (None, None)
-        kernels.rotate_heads(proj[:, :2 * Q], cos, sin, self.rotary_dim, 2 * self.heads, self.heads, self.dim, self.dim ** -0.5)
+        plan = None
+        if kernels.chunked_scan_supports(x.dtype, self.dim, self.vdim, 0, cache.state.stride(0)) and cache.state.data_ptr() % 16 == 0:
+            plan = chunk_plan(ctx)
+        rows = torch.empty((N, 2 * Q + V), dtype=x.dtype, device=x.device) if plan is not None else None
+        single = plan is None or not plan[2]                                # requests whose tokens are walked one by one
+        kernels.rotate_heads(proj[:, :2 * Q + V] if plan is not None else proj[:, :2 * Q], cos, sin, self.rotary_dim, 2 * self.heads, self.heads,
+                             self.dim, self.dim ** -0.5, typed=rows, in_place=single)
         o = torch.empty((N, V), dtype=torch.float32, device=x.device)
-        kernels.retention_scan(proj[:, :Q], proj[:, Q:2 * Q], proj[:, 2 * Q:2 * Q + V], self.decays, cache.state, 0, ctx.q_start, ctx.slots,
-                               ctx.positions, o, self.heads, self.dim, self.vdim)
+        if plan is not None:
+            kernels.chunked_scan(rows[:, Q:2 * Q], rows[:, :Q], rows[:, 2 * Q:], cache.state, 0, ctx.q_start, ctx.slots, ctx.positions, plan[0], plan[1],
+                                 o, self.heads, self.heads, self.dim, self.vdim, log_decay=self.log_decay)
+        if single:
+            kernels.retention_scan(proj[:, :Q], proj[:, Q:2 * Q], proj[:, 2 * Q:2 * Q + V], self.decays, cache.state, 0, ctx.q_start, ctx.slots,
+                                   ctx.positions, o, self.heads, self.dim, self.vdim,
+                                   max_tokens=kernels.CHUNKED_SCAN_MIN_TOKENS - 1 if plan is not None else None)
         gated = torch.empty((N, V), dtype=x.dtype, device=x.device)
         kernels.gated_group_norm(o, proj[:, 2 * Q + V:], None, gated, self.vdim, self.eps, gate_first=False)
         return linear(gated, self.w_out, out_dtype=torch.float32), None

@@ -10,7 +10,8 @@ channels, G groups of N state channels (head i reads group i // (H / G)) and inn
     y <- y * silu(z), then an RMS norm in ``norm_groups`` equal parts of the row, times ``norm``;  out = Wo y
 
 The product leaves float32; convolution, step sizes, decays, state, read-out, gate and norm are float32
-(``csrc/short_conv.cu``, ``csrc/state_space.cu``); the normed rows are rounded once to the compute type for the output
+(``csrc/short_conv.cu``, ``csrc/state_space.cu``); in bfloat16, requests of many tokens run in chunks on the tensor cores with the
+convolved x, B and C rounded to bfloat16 (``csrc/chunked_scan.cu``); the normed rows are rounded once to the compute type for the output
 product, whose result is float32 again.
 
 State of a request: one float32 vector in its slot, ``[conv piece | state piece]``. Each piece holds two copies that take
@@ -29,6 +30,20 @@ from ..ops.linear import linear
 from ..weights.source import ParamSpec
 from .base import LayerCache, Mixer, TensorGetter
 from .registry import register_mixer
+
+
+def chunk_plan(ctx):
+    """(chunks, requests, whether every request of the step is in chunks) for the step's requests of many tokens, on the device
+    (``kernels.plan_chunks``), or None where there are none. Made once per step; nothing of it in a step of single tokens."""
+    if ctx.max_q_len < kernels.CHUNKED_SCAN_MIN_TOKENS:
+        return None
+    plan = ctx.memo.get("chunk_plan")
+    if plan is None:
+        chunks, requests = kernels.plan_chunks(ctx.q_lens, kernels.CHUNKED_SCAN_MIN_TOKENS)
+        flat = torch.tensor([n for row in chunks + requests for n in row], dtype=torch.int32).pin_memory().to(ctx.device, non_blocking=True)
+        at = 2 * len(chunks)
+        plan = ctx.memo["chunk_plan"] = (flat[:at].view(-1, 2), flat[at:].view(-1, 3), len(requests) == len(ctx.q_lens))
+    return plan
 
 
 @register_mixer("ssd")
@@ -93,12 +108,23 @@ class StateSpaceDuality(Mixer):
         N, inner, C = ctx.num_tokens, self.inner, self.channels
         proj = linear(x, self.w_in, out_dtype=torch.float32)
         z, xbc, dt = proj[:, :inner], proj[:, inner:inner + C], proj[:, inner + C:]
-        mixed = torch.empty((N, C), dtype=torch.float32, device=x.device)
+        plan = None
+        if kernels.chunked_scan_supports(x.dtype, self.state, self.vdim, self.conv_entries, cache.state.stride(0)) and cache.state.data_ptr() % 16 == 0:
+            plan = chunk_plan(ctx)
+        chunked = torch.empty((N, C), dtype=x.dtype, device=x.device) if plan is not None else None
+        mixed = torch.empty((N, C), dtype=torch.float32, device=x.device) if plan is None or not plan[2] else None
         kernels.short_conv(xbc, self.conv_w, self.conv_b, cache.state, 0, ctx.q_start, ctx.slots, ctx.positions, ctx.token_request,
-                           mixed, ctx.max_q_len, silu=True)
+                           mixed, ctx.max_q_len, silu=True, out_typed=chunked)
         y = torch.empty((N, inner), dtype=torch.float32, device=x.device)
-        kernels.ssd_scan(mixed, dt, self.dt_bias, self.a_log, self.d_skip, cache.state, self.conv_entries, ctx.q_start, ctx.slots,
-                         ctx.positions, y, self.heads, self.groups, self.state, self.vdim)
+        if plan is not None:
+            GN = self.groups * self.state
+            kernels.chunked_scan(chunked[:, inner:inner + GN], chunked[:, inner + GN:], chunked[:, :inner], cache.state, self.conv_entries, ctx.q_start,
+                                 ctx.slots, ctx.positions, plan[0], plan[1], y, self.heads, self.groups, self.state, self.vdim, dt=dt,
+                                 dt_bias=self.dt_bias, a_log=self.a_log, d_skip=self.d_skip)
+        if mixed is not None:
+            kernels.ssd_scan(mixed, dt, self.dt_bias, self.a_log, self.d_skip, cache.state, self.conv_entries, ctx.q_start, ctx.slots,
+                             ctx.positions, y, self.heads, self.groups, self.state, self.vdim,
+                             max_tokens=kernels.CHUNKED_SCAN_MIN_TOKENS - 1 if plan is not None else None)
         normed = torch.empty((N, inner), dtype=x.dtype, device=x.device)
         kernels.gated_group_norm(y, z, self.norm_w, normed, inner // self.norm_groups, self.eps, gate_first=True)
         return linear(normed, self.w_out, out_dtype=torch.float32), None
