@@ -100,7 +100,7 @@ template <> __device__ __forceinline__ void rows_store4<bf16>(bf16* p, float4 v)
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
 }
 
-// A block per token. VEC: pieces of four entries (d, dv, rot multiples of 4, no rotation or the interleaved one).
+// A block per token. VEC: pieces of four entries (d, dv, rot multiples of 4, and rot / 2 too in the half-split layout).
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) capped_rows_post_kernel(const RowsPostArgs a) {
     __shared__ float scratch[32];
@@ -152,7 +152,15 @@ __global__ void __launch_bounds__(256) capped_rows_post_kernel(const RowsPostArg
             float4 v = *reinterpret_cast<const float4*>(row + i);
             const float4 w = *reinterpret_cast<const float4*>((is_q ? a.qw : a.kw) + j);
             v = make_float4(v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w);
-            if (c < a.rot) {
+            if (c < a.rot && !a.interleaved) {     // the piece of the pairs' other entries lies rot / 2 before or behind
+                const bool first = c < half;
+                const int at = first ? c : c - half, to = first ? half : -half;
+                const float4 ov = *reinterpret_cast<const float4*>(row + i + to), ow = *reinterpret_cast<const float4*>((is_q ? a.qw : a.kw) + j + to);
+                const float4 co = *reinterpret_cast<const float4*>(cs + at), si = *reinterpret_cast<const float4*>(sn + at);
+                const float fs = first ? -f : f;
+                v = make_float4(v.x * co.x + ov.x * fs * ow.x * si.x, v.y * co.y + ov.y * fs * ow.y * si.y, v.z * co.z + ov.z * fs * ow.z * si.z,
+                                v.w * co.w + ov.w * fs * ow.w * si.w);
+            } else if (c < a.rot) {
                 const float2 co = *reinterpret_cast<const float2*>(cs + (c >> 1)), si = *reinterpret_cast<const float2*>(sn + (c >> 1));
                 v = make_float4(v.x * co.x - v.y * si.x, v.y * co.x + v.x * si.x, v.z * co.y - v.w * si.y, v.w * co.y + v.z * si.y);
             }
@@ -328,7 +336,7 @@ LLMP_API int llmp_capped_rows_post(const float* proj, long proj_t, const float* 
     RowsPostArgs a;
     a.proj = proj; a.proj_t = proj_t; a.qw = qw; a.kw = kw; a.eps = eps; a.cos_t = cos_t; a.sin_t = sin_t; a.rot = rot; a.interleaved = interleaved;
     a.q_out = q_out; a.q_out_t = q_out_t; a.slots = slots; a.pages = pages; a.page_size = page_size; a.H = H; a.G = G; a.d = d; a.dv = dv; a.v_at = v_at;
-    const bool vec = d % 4 == 0 && dv % 4 == 0 && rot % 4 == 0 && (rot == 0 || interleaved) && proj_t % 4 == 0 && v_at % 4 == 0 && q_out_t % 4 == 0 &&
+    const bool vec = d % 4 == 0 && dv % 4 == 0 && rot % 4 == 0 && (rot == 0 || interleaved || rot % 8 == 0) && proj_t % 4 == 0 && v_at % 4 == 0 && q_out_t % 4 == 0 &&
                      ((size_t)proj | (size_t)qw | (size_t)kw | (size_t)cos_t | (size_t)sin_t | (size_t)q_out | (size_t)pages) % 16 == 0;
     void (*kernel)(const RowsPostArgs) = dtype == LLMP_F32 ? (vec ? capped_rows_post_kernel<float, true> : capped_rows_post_kernel<float, false>)
                                                            : (vec ? capped_rows_post_kernel<bf16, true> : capped_rows_post_kernel<bf16, false>);

@@ -150,6 +150,65 @@ __global__ void short_conv_parallel_kernel(const ConvArgs a, const int N) {
     }
 }
 
+// The same with four channels a thread in 16-byte accesses, for K = 2, 3 or 4 taps.
+template <int K>
+__global__ void __launch_bounds__(128) short_conv_by_4_kernel(const ConvArgs a, const int N) {
+    pdl_wait();
+    pdl_trigger();
+    const int t0 = blockIdx.x * CONV_TILE_TOKENS;
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+    if (c >= a.C) return;
+    auto load = [&](const float* p) { return *reinterpret_cast<const float4*>(p); };
+    float4 tap[K], w[K - 1];
+#pragma unroll
+    for (int j = 0; j < K; ++j)
+        tap[j] = make_float4(load_as_float(a.taps, a.taps_bf16, (size_t)c * K + j), load_as_float(a.taps, a.taps_bf16, (size_t)(c + 1) * K + j),
+                             load_as_float(a.taps, a.taps_bf16, (size_t)(c + 2) * K + j), load_as_float(a.taps, a.taps_bf16, (size_t)(c + 3) * K + j));
+    float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (a.bias) b = make_float4(load_as_float(a.bias, a.bias_bf16, c), load_as_float(a.bias, a.bias_bf16, c + 1), load_as_float(a.bias, a.bias_bf16, c + 2),
+                                load_as_float(a.bias, a.bias_bf16, c + 3));
+    const size_t base2 = conv_out2_base(a, c);
+    const int t1 = min(t0 + CONV_TILE_TOKENS, N);
+    int r_prev = -1;
+#pragma unroll 4
+    for (int t = t0; t < t1; ++t) {
+        const float4 xin = load(a.x + (size_t)t * a.x_t + c);
+        const int r = a.token_request[t];
+        if (r != r_prev) {
+            r_prev = r;
+            const int begin = a.q_start[r];
+            const int p0 = a.positions[begin];
+            const float* rd = a.state + (size_t)a.slots[r] * a.state_slot + ((p0 + 1) & 1) * a.state_half;
+#pragma unroll
+            for (int j = 0; j < K - 1; ++j) {
+                const int at = t - (K - 1) + j;
+                w[j] = at >= begin ? load(a.x + (size_t)at * a.x_t + c) : load(rd + (size_t)(K - 1 + at - begin) * a.C + c);
+            }
+        }
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < K; ++j) {
+            const float4 u = j < K - 1 ? w[j < K - 1 ? j : 0] : xin;
+            v = make_float4(fmaf(u.x, tap[j].x, v.x), fmaf(u.y, tap[j].y, v.y), fmaf(u.z, tap[j].z, v.z), fmaf(u.w, tap[j].w, v.w));
+        }
+        v = make_float4(conv_act(v.x + b.x, xin.x, a.act), conv_act(v.y + b.y, xin.y, a.act), conv_act(v.z + b.z, xin.z, a.act),
+                        conv_act(v.w + b.w, xin.w, a.act));
+        if (a.out) *reinterpret_cast<float4*>(a.out + (size_t)t * a.out_t + c) = v;
+        if (a.out2) {
+            const size_t at = base2 + (size_t)t * a.out2_t;
+            if (a.out2_bf16) {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+                *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out2) + at) = make_uint2(*reinterpret_cast<const unsigned*>(&lo),
+                                                                                             *reinterpret_cast<const unsigned*>(&hi));
+            } else {
+                *reinterpret_cast<float4*>(reinterpret_cast<float*>(a.out2) + at) = v;
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < K - 1; ++j) w[j] = j + 1 < K - 1 ? w[j + 1 < K - 1 ? j + 1 : 0] : xin;
+    }
+}
+
 __global__ void short_conv_state_kernel(const ConvArgs a) {
     const int r = blockIdx.x;
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -203,7 +262,14 @@ LLMP_API int llmp_short_conv(const float* x, long x_t, const void* taps, int tap
         llmp_launch_dependent(short_conv_serial_kernel, dim3(R, col_blocks), dim3(threads), 0, stream, a);
         return llmp_check_launch("short_conv");
     }
-    short_conv_parallel_kernel<<<dim3((N + CONV_TILE_TOKENS - 1) / CONV_TILE_TOKENS, col_blocks), threads, 0, stream>>>(a, N);
+    const bool by4 = C % 4 == 0 && x_t % 4 == 0 && state_slot % 4 == 0 && state_half % 4 == 0 && ((uintptr_t)x | (uintptr_t)state) % 16 == 0 &&
+                     (!out || (out_t % 4 == 0 && (uintptr_t)out % 16 == 0)) &&
+                     (!out2 || (a.out2_split % 4 == 0 && out2_t % 4 == 0 && out2_block % 4 == 0 && (uintptr_t)out2 % (a.out2_bf16 ? 8 : 16) == 0));
+    const dim3 grid4((N + CONV_TILE_TOKENS - 1) / CONV_TILE_TOKENS, (C / 4 + threads - 1) / threads);
+    if (by4 && K == 2) llmp_launch_dependent(short_conv_by_4_kernel<2>, grid4, dim3(threads), 0, stream, a, N);
+    else if (by4 && K == 3) llmp_launch_dependent(short_conv_by_4_kernel<3>, grid4, dim3(threads), 0, stream, a, N);
+    else if (by4 && K == 4) llmp_launch_dependent(short_conv_by_4_kernel<4>, grid4, dim3(threads), 0, stream, a, N);
+    else short_conv_parallel_kernel<<<dim3((N + CONV_TILE_TOKENS - 1) / CONV_TILE_TOKENS, col_blocks), threads, 0, stream>>>(a, N);
     if (K > 1) short_conv_state_kernel<<<dim3(R, col_blocks), threads, 0, stream>>>(a);
     return llmp_check_launch("short_conv (parallel)");
 }

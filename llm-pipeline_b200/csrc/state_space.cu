@@ -203,6 +203,68 @@ __global__ void gated_group_norm_kernel(const NormArgs a) {
     }
 }
 
+__device__ __forceinline__ float gn_gate(const NormArgs& a, float y, float z) { return a.mode == 0 ? y * (z / (1.f + expf(-z))) : y; }
+__device__ __forceinline__ float gn_out(const NormArgs& a, float v, float z, float inv, float w) {
+    if (a.mode == 0) return v * inv * w;
+    return v * inv * (a.mode == 1 ? w : z) * (1.f / (1.f + expf(-z)));
+}
+
+// The same in 16-byte pieces with the group in registers: NP pieces of four entries a lane.
+template <typename T, bool TEAM, int NP>
+__global__ void gated_group_norm_rows_kernel(const NormArgs a) {
+    __shared__ float scratch[32];
+    pdl_wait();
+    pdl_trigger();
+    const int groups = a.W / a.gs, g4 = a.gs >> 2;
+    const long item = TEAM ? (long)blockIdx.x : (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= (long)a.tokens * groups) return;
+    const int lane = TEAM ? threadIdx.x : threadIdx.x & 31;
+    const int step = TEAM ? blockDim.x : 32;
+    const int t = (int)(item / groups), c0 = (int)(item % groups) * a.gs;
+    const float4* y = reinterpret_cast<const float4*>(a.y + (size_t)t * a.y_t + c0);
+    const float4* gate = reinterpret_cast<const float4*>(a.gate + (size_t)t * a.gate_t + c0);
+    float4 v[NP], z[NP];
+    float ss = 0.f;
+#pragma unroll
+    for (int p = 0; p < NP; ++p) {
+        const int i = lane + p * step;
+        v[p] = z[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < g4) { v[p] = y[i]; z[p] = gate[i]; }
+    }
+#pragma unroll
+    for (int p = 0; p < NP; ++p) {
+        v[p] = make_float4(gn_gate(a, v[p].x, z[p].x), gn_gate(a, v[p].y, z[p].y), gn_gate(a, v[p].z, z[p].z), gn_gate(a, v[p].w, z[p].w));
+        ss = fmaf(v[p].x, v[p].x, fmaf(v[p].y, v[p].y, fmaf(v[p].z, v[p].z, fmaf(v[p].w, v[p].w, ss))));
+    }
+    ss = TEAM ? block_sum(ss, scratch) : warp_sum(ss);
+    const float inv = 1.f / sqrtf(ss / (float)a.gs + a.eps);
+    T* out = reinterpret_cast<T*>(a.out) + (size_t)t * a.out_t + c0;
+#pragma unroll
+    for (int p = 0; p < NP; ++p) {
+        const int i = lane + p * step;
+        if (i >= g4) continue;
+        float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (a.mode != 2) w = reinterpret_cast<const float4*>(a.weight + (a.mode == 0 ? c0 : 0))[i];
+        const float o0 = gn_out(a, v[p].x, z[p].x, inv, w.x), o1 = gn_out(a, v[p].y, z[p].y, inv, w.y);
+        const float o2 = gn_out(a, v[p].z, z[p].z, inv, w.z), o3 = gn_out(a, v[p].w, z[p].w, inv, w.w);
+        if constexpr (sizeof(T) == 4) reinterpret_cast<float4*>(out)[i] = make_float4(o0, o1, o2, o3);
+        else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(o0, o1), hi = __floats2bfloat162_rn(o2, o3);
+            reinterpret_cast<uint2*>(out)[i] = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+        }
+    }
+}
+
+template <typename T> void launch_norm_rows(const NormArgs& a, long items, cudaStream_t stream) {
+    // the form depends on the group's size alone
+    const int g4 = a.gs / 4, warps = 8;
+    const dim3 per_warp((unsigned)((items + warps - 1) / warps)), per_block((unsigned)items);
+    if (g4 <= 32) llmp_launch_dependent(gated_group_norm_rows_kernel<T, false, 1>, per_warp, dim3(32 * warps), 0, stream, a);
+    else if (g4 <= 64) llmp_launch_dependent(gated_group_norm_rows_kernel<T, false, 2>, per_warp, dim3(32 * warps), 0, stream, a);
+    else if (g4 <= 256) llmp_launch_dependent(gated_group_norm_rows_kernel<T, true, 2>, per_block, dim3(128), 0, stream, a);
+    else llmp_launch_dependent(gated_group_norm_rows_kernel<T, true, 4>, per_block, dim3(512), 0, stream, a);
+}
+
 }  // namespace
 
 static int launch_scan(const ScanArgs& a, int R, cudaStream_t stream) {
@@ -283,6 +345,12 @@ LLMP_API int llmp_gated_group_norm(const float* y, long y_t, const float* gate, 
     a.y = y; a.y_t = y_t; a.gate = gate; a.gate_t = gate_t; a.weight = weight; a.out = out; a.out_t = out_t;
     a.tokens = tokens; a.W = W; a.gs = gs; a.mode = mode; a.eps = eps;
     const long items = (long)tokens * (W / gs);
+    if (gs % 4 == 0 && gs <= 8192 && y_t % 4 == 0 && gate_t % 4 == 0 && out_t % 4 == 0 &&
+        ((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight) % 16 == 0 && (uintptr_t)out % (out_dtype == LLMP_BF16 ? 8 : 16) == 0) {
+        if (out_dtype == LLMP_BF16) launch_norm_rows<bf16>(a, items, stream);
+        else launch_norm_rows<float>(a, items, stream);
+        return llmp_check_launch("gated_group_norm");
+    }
     if (gs >= 512) {                     // a block per group; the choice depends on the group's size alone
         const int threads = gs >= 2048 ? 512 : 256;
         if (out_dtype == LLMP_BF16) gated_group_norm_kernel<bf16, true><<<(unsigned)items, threads, 0, stream>>>(a);

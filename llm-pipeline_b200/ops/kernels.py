@@ -94,6 +94,8 @@ _SIGNATURES = {
     "llmp_ssd_scan": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _P],
     "llmp_retention_scan": [_P, _P, _P, _L, _P, _P, _L, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P],
     "llmp_rotate_heads": [_P, _L, _P, _L, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
+    "llmp_ssd_step": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _L, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P],
+    "llmp_retention_step": [_P, _P, _P, _P, _L, _P, _P, _I, _F, _P, _F, _P, _L, _L, _P, _P, _P, _I, _L, _I, _I, _I, _I, _P],
     "llmp_chunked_scan": [_P, _P, _P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _L, _P, _P, _P, _P, _I, _P, _I, _P, _P, _P, _L, _I, _I, _I, _I, _P],
     "llmp_stream_step": [_P, _L, _L, _P, _P, _I, _P, _F, _F, _P, _I, _P, _F, _F, _P, _P, _P, _P, _P, _I, _F, _P, _I, _P, _I, _I, _I, _P],
     "llmp_gated_group_norm": [_P, _L, _P, _L, _P, _P, _I, _L, _I, _I, _I, _I, _F, _P],
@@ -1361,6 +1363,53 @@ def retention_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
     _call("llmp_retention_scan", _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), ptr, slot_stride, half, _ptr(q_start), _ptr(slots),
           _ptr(positions), _ptr(y), y.stride(0), slots.numel(), heads, dim, vdim, _ALL_TOKENS if max_tokens is None else int(max_tokens), _stream())
     return y
+
+
+def state_step_supports(state: torch.Tensor, offset: int, state_size: int, vdim: int) -> bool:
+    """Whether the kernels for one token per request take this state (columns in 16-byte pieces)."""
+    return (vdim % 4 == 0 and 4 <= vdim <= 1024 and state_size <= 4096 and offset % 4 == 0 and (state_size * vdim) % 4 == 0 and
+            state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0)
+
+
+def ssd_step(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, d_skip: torch.Tensor, state: torch.Tensor,
+             state_offset: int, slots: torch.Tensor, positions: torch.Tensor, y: torch.Tensor, heads: int, groups: int, state_size: int,
+             vdim: int) -> torch.Tensor:
+    """``ssd_scan`` for a step in which every request brings one token: row r is request r (csrc/state_step.cu)."""
+    R = xbc.shape[0]
+    _need(xbc.dtype == torch.float32 and xbc.stride(1) == 1 and xbc.shape[1] == heads * vdim + 2 * groups * state_size,
+          "ssd_step: x | B | C has the wrong width")
+    _need(dt.dtype == torch.float32 and dt.stride(1) == 1 and dt.shape == (R, heads), "ssd_step: dt must be float32 [requests, heads]")
+    _need(y.dtype == torch.float32 and y.stride(1) == 1 and y.shape == (R, heads * vdim), "ssd_step: y has the wrong shape")
+    for t in (dt_bias, a_log, d_skip):
+        _need(t.dtype == torch.float32 and t.numel() == heads and t.is_contiguous(), "ssd_step takes float32 vectors of one entry per head")
+    _i32(slots, "slots")
+    _i32(positions, "positions")
+    ptr, slot_stride, half = _state_views(state, state_offset, heads * state_size * vdim, "ssd_step")
+    _call("llmp_ssd_step", _ptr(xbc), xbc.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), ptr, slot_stride, half,
+          _ptr(slots), _ptr(positions), _ptr(y), y.stride(0), R, heads, groups, state_size, vdim, _stream())
+    return y
+
+
+def retention_step(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
+                   rot: int, k_scale: float, decay: torch.Tensor, eps: float, state: torch.Tensor, state_offset: int, slots: torch.Tensor,
+                   positions: torch.Tensor, out: torch.Tensor, heads: int, dim: int, vdim: int) -> torch.Tensor:
+    """Retention for a step in which every request brings one token, from the input product's rows to the gated rows
+    (csrc/state_step.cu): q and k turned and k scaled, the state moved on and read, each head's row divided by its root mean
+    square and multiplied by silu(gate). ``q`` .. ``gate``: float32 views with one stride; ``out`` [requests, heads vdim]."""
+    R = q.shape[0]
+    _need(all(t.dtype == torch.float32 and t.stride(1) == 1 and t.stride(0) == q.stride(0) for t in (q, k, v, gate)), "retention_step takes float32 rows")
+    _need(q.shape == k.shape == (R, heads * dim) and v.shape == gate.shape == out.shape == (R, heads * vdim) and out.stride(1) == 1,
+          "retention_step: rows have the wrong shape")
+    _need(decay.dtype == torch.float32 and decay.is_contiguous() and decay.shape == (2, heads), "retention_step: decays must be float32 [2, heads]")
+    _need(rot == 0 or (cos.dtype == sin.dtype == torch.float32 and cos.is_contiguous() and sin.is_contiguous() and
+                       cos.shape == sin.shape == (R, rot // 2)), "retention_step: rotary tables have the wrong shape")
+    _i32(slots, "slots")
+    _i32(positions, "positions")
+    ptr, slot_stride, half = _state_views(state, state_offset, heads * dim * vdim, "retention_step")
+    _call("llmp_retention_step", _ptr(q), _ptr(k), _ptr(v), _ptr(gate), q.stride(0), _ptr(cos), _ptr(sin), int(rot), float(k_scale), _ptr(decay),
+          float(eps), ptr, slot_stride, half, _ptr(slots), _ptr(positions), _ptr(out), dtype_code(out.dtype), out.stride(0), R, heads, dim, vdim,
+          _stream())
+    return out
 
 
 CHUNKED_SCAN_TOKENS = 128            # csrc/chunked_scan.cu: tokens of a chunk

@@ -86,6 +86,13 @@ class Retention(Mixer):
         N, Q, V = ctx.num_tokens, self.qk_size, self.v_size
         proj = linear(x, self.w_in, out_dtype=torch.float32)                # [N, q | k | v | gate]
         cos, sin = ctx.position_tables[self.position] if self.rotary_dim else (None, None)
+        gate = proj[:, 2 * Q + V:]
+        gated = torch.empty((N, V), dtype=x.dtype, device=x.device)
+        if ctx.max_q_len == 1 and kernels.state_step_supports(cache.state, 0, self.dim, self.vdim):
+            # one token a request: rotation, state, norm and gate in one kernel
+            kernels.retention_step(proj[:, :Q], proj[:, Q:2 * Q], proj[:, 2 * Q:2 * Q + V], gate, cos, sin, self.rotary_dim, self.dim ** -0.5,
+                                   self.decays, self.eps, cache.state, 0, ctx.slots, ctx.positions, gated, self.heads, self.dim, self.vdim)
+            return linear(gated, self.w_out, out_dtype=torch.float32), None
         plan = None
         if kernels.chunked_scan_supports(x.dtype, self.dim, self.vdim, 0, cache.state.stride(0)) and cache.state.data_ptr() % 16 == 0:
             plan = chunk_plan(ctx)
@@ -101,6 +108,5 @@ class Retention(Mixer):
             kernels.retention_scan(proj[:, :Q], proj[:, Q:2 * Q], proj[:, 2 * Q:2 * Q + V], self.decays, cache.state, 0, ctx.q_start, ctx.slots,
                                    ctx.positions, o, self.heads, self.dim, self.vdim,
                                    max_tokens=kernels.CHUNKED_SCAN_MIN_TOKENS - 1 if plan is not None else None)
-        gated = torch.empty((N, V), dtype=x.dtype, device=x.device)
-        kernels.gated_group_norm(o, proj[:, 2 * Q + V:], None, gated, self.vdim, self.eps, gate_first=False)
+        kernels.gated_group_norm(o, gate, None, gated, self.vdim, self.eps, gate_first=False)
         return linear(gated, self.w_out, out_dtype=torch.float32), None

@@ -103,6 +103,7 @@ class StateSpaceDuality(Mixer):
                                                               for n in ("dt_bias", "A_log", "D", "norm"))
 
     def forward(self, x, ctx, cache: LayerCache):
+        # (what a kernel is chosen by does not change while a captured step is replayed: row strides and the step's shape)
         if cache.state is None:
             raise RuntimeError("the state-space mixer needs its state slots")
         N, inner, C = ctx.num_tokens, self.inner, self.channels
@@ -121,7 +122,10 @@ class StateSpaceDuality(Mixer):
             kernels.chunked_scan(chunked[:, inner:inner + GN], chunked[:, inner + GN:], chunked[:, :inner], cache.state, self.conv_entries, ctx.q_start,
                                  ctx.slots, ctx.positions, plan[0], plan[1], y, self.heads, self.groups, self.state, self.vdim, dt=dt,
                                  dt_bias=self.dt_bias, a_log=self.a_log, d_skip=self.d_skip)
-        if mixed is not None:
+        if ctx.max_q_len == 1 and kernels.state_step_supports(cache.state, self.conv_entries, self.state, self.vdim):
+            kernels.ssd_step(mixed, dt, self.dt_bias, self.a_log, self.d_skip, cache.state, self.conv_entries, ctx.slots, ctx.positions, y, self.heads,
+                             self.groups, self.state, self.vdim)
+        elif mixed is not None:
             kernels.ssd_scan(mixed, dt, self.dt_bias, self.a_log, self.d_skip, cache.state, self.conv_entries, ctx.q_start, ctx.slots,
                              ctx.positions, y, self.heads, self.groups, self.state, self.vdim,
                              max_tokens=kernels.CHUNKED_SCAN_MIN_TOKENS - 1 if plan is not None else None)

@@ -252,7 +252,68 @@ def test_the_rotated_rows_in_bfloat16(monkeypatch):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads, dim", [(3, 16), (2, 20), (1, 100), (3, 7), (2, 600)])
+@pytest.mark.parametrize("sizes", [(3, 16, 20, 8), (2, 20, 8, 6), (1, 5, 64, 4), (2, 128, 128, 128), (5, 33, 48, 0), (1, 256, 512, 64), (2, 300, 4, 2)], ids=str)
+def test_one_token_a_request_through_retention_alone(dtype, sizes):
+    """From the input product's rows to the gated rows, token by token for requests that start at different times."""
+    from llm_pipeline_b200.ops import kernels
+    heads, dim, vdim, rot = sizes
+    gen = torch.Generator().manual_seed(dim * vdim)
+    Q, V, base, eps = heads * dim, heads * vdim, 40.0, 1e-5
+    decay = torch.tensor(([0.997, 0.0, 1.0, 0.8, 0.95] * 2)[:heads], dtype=torch.float64)
+    decays = torch.stack([decay.float(), (decay - decay.float().double()).float()]).to(DEV)
+    rows = {s: torch.randn(n, 2 * Q + 2 * V, generator=gen) for s, n in ((2, 12), (0, 9))}
+    want = {}
+    for s, x in rows.items():
+        q = plain.rotate(x[:, :Q].double().view(-1, heads, dim), {"base": base, "dims": rot})
+        k = plain.rotate(x[:, Q:2 * Q].double().view(-1, heads, dim), {"base": base, "dims": rot}) * 0.3
+        o, _ = plain.retention_scan(q, k, x[:, 2 * Q:2 * Q + V].double().view(-1, heads, vdim), decay)
+        want[s] = plain.rms(o, eps).reshape(-1, V) * plain.silu(x[:, 2 * Q + V:].double())
+    offset, half = 4, heads * dim * vdim
+    state = torch.full((4, offset + 2 * half + (-2 * half) % 4), 7.0, device=DEV)
+    state[[0, 2]] = 0.0
+    assert kernels.state_step_supports(state, offset, dim, vdim)
+    inv = torch.tensor([base ** (-2.0 * i / rot) for i in range(rot // 2)] or [1.0], device=DEV)
+    for t in range(12):
+        live = [s for s, start in ((2, 0), (0, 3)) if start <= t and t - start < rows[s].shape[0]]
+        at = [t if s == 2 else t - 3 for s in live]
+        x = torch.stack([rows[s][i] for s, i in zip(live, at)]).to(DEV)
+        positions, cos, sin = _i32(at), None, None
+        if rot:
+            cos, sin = (torch.empty(len(live), rot // 2, device=DEV) for _ in range(2))
+            kernels.rope_tables(positions, inv, 1.0, cos, sin)
+        out = torch.empty(len(live), V, device=DEV, dtype=dtype)
+        kernels.retention_step(x[:, :Q], x[:, Q:2 * Q], x[:, 2 * Q:2 * Q + V], x[:, 2 * Q + V:], cos, sin, rot, 0.3, decays, eps, state, offset,
+                               _i32(live), positions, out, heads, dim, vdim)
+        assert _rel(out, torch.stack([want[s][i] for s, i in zip(live, at)])) < (2e-5 if dtype == torch.float32 else 1e-2), t
+    assert (state[[1, 3]] == 7.0).all() and (state[[0, 2], :offset] == 0.0).all()
+
+
+@pytest.mark.parametrize("sizes", [(4, 2, 24, 16), (3, 1, 7, 12), (2, 2, 128, 128), (6, 3, 300, 64), (1, 1, 16, 1024)], ids=str)
+def test_one_token_a_request_through_the_state_space_alone(sizes):
+    """A prompt through the token-by-token kernel, then single tokens; the state goes from one to the other and back."""
+    from llm_pipeline_b200.ops import kernels
+    heads, groups, N, P = sizes
+    gen = torch.Generator().manual_seed(N * P)
+    C = heads * P + 2 * groups * N
+    n = 15
+    x, dt = torch.randn(n, C, generator=gen), torch.randn(n, heads, generator=gen)
+    bias, a_log, skip = (torch.randn(heads, generator=gen) for _ in range(3))
+    want = plain.ssd_scan(x[:, :heads * P].double().view(n, heads, P), x[:, heads * P:heads * P + groups * N].double().view(n, groups, N),
+                          x[:, heads * P + groups * N:].double().view(n, groups, N), torch.nn.functional.softplus(dt.double() + bias.double()),
+                          a_log.double(), skip.double()).reshape(n, -1)
+    xd, dd, args = x.to(DEV), dt.to(DEV), [t.to(DEV) for t in (bias, a_log, skip)]
+    state = torch.zeros(3, 4 + 2 * heads * N * P, device=DEV)
+    y = torch.full((n, heads * P), float("nan"), device=DEV)
+    for lo, hi in [(0, 4)] + [(t, t + 1) for t in range(4, 11)] + [(11, 14), (14, 15)]:
+        if hi - lo == 1:
+            kernels.ssd_step(xd[lo:hi], dd[lo:hi], *args, state, 4, _i32([1]), _i32([lo]), y[lo:hi], heads, groups, N, P)
+        else:
+            kernels.ssd_scan(xd[lo:hi], dd[lo:hi], *args, state, 4, _i32([0, hi - lo]), _i32([1]), _i32(list(range(lo, hi))), y[lo:hi], heads, groups, N, P)
+    assert _rel(y, want) < 5e-6 and (state[[0, 2]] == 0.0).all()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads, dim", [(3, 16), (2, 20), (1, 100), (3, 7), (2, 600), (1, 2048), (2, 200), (1, 9000)])
 def test_heads_norm_and_silu_gate_alone(dtype, heads, dim):
     from llm_pipeline_b200.ops import kernels
     gen = torch.Generator().manual_seed(dim)
