@@ -1027,11 +1027,14 @@ def zavizen_work(z, tokens, keys_per_token, decode, requests=1):
     # expert sum and a shared expert stand beside each other)
     work["stream_step"] = (tokens * D * (2 * L * (8 * S + 2) + 4 * (2 * L + par + moe)), 0.0)
     work["capped_rows_post"] = (par * tokens * (H + 2 * G) * d * (4 + 2), 0.0)
-    work["short_conv"] = (ssm * tokens * channels * 8, 0.0)
-    # queries, keys and values in, read-outs out, every request's state read and written once
-    work["retention_scan"] = (par * (tokens * Hr * 4 * (2 * dr + 2 * vr) + requests * Hr * dr * vr * 8), 0.0)
-    work["ssd_scan"] = (ssm * (tokens * 4 * (channels + inner) + requests * z["ssm_heads"] * z["state"] * z["ssm_vdim"] * 8), 0.0)
-    work["rotate_heads"] = (par * tokens * 2 * Hr * dr * 8, 0.0)
+    work["short_conv"] = (ssm * tokens * channels * (8 if decode else 6), 0.0)
+    # one token a request: rows in float32, every request's state read and written once
+    work["retention_step"] = (par * (tokens * Hr * (4 * (2 * dr + 2 * vr) + 2 * vr) + requests * Hr * dr * vr * 8), 0.0)
+    work["ssd_step"] = (ssm * (tokens * 4 * (channels + inner) + requests * z["ssm_heads"] * z["state"] * z["ssm_vdim"] * 8), 0.0)
+    # chunks: bfloat16 rows in, float32 read-outs out, the states in and out; nothing of what passes through scratch
+    work["chunked_scan"] = (par * (tokens * Hr * (2 * (2 * dr + vr) + 4 * vr) + requests * Hr * dr * vr * 8) +
+                            ssm * (tokens * (2 * channels + 4 * inner) + requests * z["ssm_heads"] * z["state"] * z["ssm_vdim"] * 8), 0.0)
+    work["rotate_heads"] = (par * tokens * Hr * (2 * dr + vr) * 6, 0.0)
     work["gated_group_norm"] = (tokens * (ssm * inner + par * Hr * vr) * (4 + 4 + 2), 0.0)
     work["swiglu"] = (tokens * 6 * ((L - moe) * z["ff"] + moe * z["shared_ff"]), 0.0)
     if decode:

@@ -251,6 +251,10 @@ class Mixer(Part):
     def forward(self, x: torch.Tensor, ctx, cache: LayerCache) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         raise NotImplementedError
 
+    # Optional: a mixer whose input is read by one product with a float32 result alone may hold that product's matrix as
+    # ``w_in`` and offer ``forward_from(proj, ctx, cache)``, which goes on from the product's rows (any stride between them);
+    # mixers that read the same input can then share one product.
+
 
 class FeedForward(Part):
     def forward(self, x: torch.Tensor, ctx) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:

@@ -182,13 +182,15 @@ class CappedAttention(Mixer):
             self.sinks = torch.full((H,), float(self.sink), dtype=torch.float32, device=device)
 
     def forward(self, x, ctx, cache: LayerCache):
+        return self.forward_from(linear(x, self.w_in, out_dtype=torch.float32), ctx, cache)         # [N, q | k | v | gate]
+
+    def forward_from(self, proj, ctx, cache: LayerCache):
         if cache.pages is None or cache.group is None:
             raise RuntimeError("the capped attention mixer needs the pages of its cache")
         N = ctx.num_tokens
-        proj = linear(x, self.w_in, out_dtype=torch.float32)               # [N, q | k | v | gate]
         sizes = {"q": self.q_size, "k": self.k_size, "v": self.v_size}
         width = sum(sizes[n] for n in self._projections())
-        q = torch.empty((N, self.q_size), dtype=x.dtype, device=x.device)
+        q = torch.empty((N, self.q_size), dtype=ctx.dtype, device=proj.device)
         writes = cache.writes and self.own_rows
         pages, slots = (cache.pages, ctx.slot_mapping[cache.group]) if writes else (None, None)
         if self.row_norm_eps is None:
@@ -199,11 +201,11 @@ class CappedAttention(Mixer):
             v_at = self.q_size + (0 if self.values_are_keys else self.k_size)
             kernels.capped_rows_post(proj, self.q_norm, self.k_norm, self.row_norm_eps, cos, sin, self.rotary_dim, self.interleaved, q, slots,
                                      pages, v_at, self.num_heads, self.num_kv_heads, self.dim, self.vdim)
-        out = torch.empty((N, self.o_size), dtype=x.dtype, device=x.device)
+        out = torch.empty((N, self.o_size), dtype=ctx.dtype, device=proj.device)
         gate = proj[:, width:] if self.gate else None
         tables = ctx.block_tables[cache.group]
         sizes = (self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.window or 0, self.keep_first, self.scale, self.softcap)
-        if kernels.capped_mma_supports(x.dtype, self.dim, self.vdim) and (width % 2 == 0 or self.gate is not True):
+        if kernels.capped_mma_supports(ctx.dtype, self.dim, self.vdim) and (width % 2 == 0 or self.gate is not True):
             # bfloat16 and sizes the tensor-core kernel has instances of: prompts in tiles of 64 rows (token, head of a group),
             # single tokens with the four warps of a block sharing the keys
             tile_req, tile_tok0 = self._tiles(ctx, kernels.capped_mma_tokens_per_tile(self.num_heads, self.num_kv_heads))

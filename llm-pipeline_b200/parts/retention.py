@@ -81,26 +81,28 @@ class Retention(Mixer):
         self.log_decay = torch.log(exact).clamp(min=-1e30).float().to(self.w_out.device)
 
     def forward(self, x, ctx, cache: LayerCache):
+        return self.forward_from(linear(x, self.w_in, out_dtype=torch.float32), ctx, cache)         # [N, q | k | v | gate]
+
+    def forward_from(self, proj, ctx, cache: LayerCache):
         if cache.state is None:
             raise RuntimeError("the retention mixer needs its state slots")
         N, Q, V = ctx.num_tokens, self.qk_size, self.v_size
-        proj = linear(x, self.w_in, out_dtype=torch.float32)                # [N, q | k | v | gate]
         cos, sin = ctx.position_tables[self.position] if self.rotary_dim else (None, None)
         gate = proj[:, 2 * Q + V:]
-        gated = torch.empty((N, V), dtype=x.dtype, device=x.device)
+        gated = torch.empty((N, V), dtype=ctx.dtype, device=proj.device)
         if ctx.max_q_len == 1 and kernels.state_step_supports(cache.state, 0, self.dim, self.vdim):
             # one token a request: rotation, state, norm and gate in one kernel
             kernels.retention_step(proj[:, :Q], proj[:, Q:2 * Q], proj[:, 2 * Q:2 * Q + V], gate, cos, sin, self.rotary_dim, self.dim ** -0.5,
                                    self.decays, self.eps, cache.state, 0, ctx.slots, ctx.positions, gated, self.heads, self.dim, self.vdim)
             return linear(gated, self.w_out, out_dtype=torch.float32), None
         plan = None
-        if kernels.chunked_scan_supports(x.dtype, self.dim, self.vdim, 0, cache.state.stride(0)) and cache.state.data_ptr() % 16 == 0:
+        if kernels.chunked_scan_supports(ctx.dtype, self.dim, self.vdim, 0, cache.state.stride(0)) and cache.state.data_ptr() % 16 == 0:
             plan = chunk_plan(ctx)
-        rows = torch.empty((N, 2 * Q + V), dtype=x.dtype, device=x.device) if plan is not None else None
+        rows = torch.empty((N, 2 * Q + V), dtype=ctx.dtype, device=proj.device) if plan is not None else None
         single = plan is None or not plan[2]                                # requests whose tokens are walked one by one
         kernels.rotate_heads(proj[:, :2 * Q + V] if plan is not None else proj[:, :2 * Q], cos, sin, self.rotary_dim, 2 * self.heads, self.heads,
                              self.dim, self.dim ** -0.5, typed=rows, in_place=single)
-        o = torch.empty((N, V), dtype=torch.float32, device=x.device)
+        o = torch.empty((N, V), dtype=torch.float32, device=proj.device)
         if plan is not None:
             kernels.chunked_scan(rows[:, Q:2 * Q], rows[:, :Q], rows[:, 2 * Q:], cache.state, 0, ctx.q_start, ctx.slots, ctx.positions, plan[0], plan[1],
                                  o, self.heads, self.heads, self.dim, self.vdim, log_decay=self.log_decay)

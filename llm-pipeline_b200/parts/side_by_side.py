@@ -5,7 +5,8 @@ any two registered mixers can stand beside each other. What they ask of the cach
 member may keep pages (the layer has one page group), and the members' states lie one after the other in the request's
 state vector, each member seeing its own column range. The sum ``left_scale * left + right_scale * right`` is float32. With
 ``out_norm_eps`` each member's result first passes an RMS norm over its row with a weight of its own (``out_norms``: the two
-names); a block that takes addends gets both results with their norms and leaves the work to the kernel that adds them."""
+names). Where both members read their input through one product each and can go on from its rows (``Mixer.forward_from``), the
+two products are one. A block that takes addends gets both results with their norms and leaves the work to the kernel that adds them."""
 
 from __future__ import annotations
 
@@ -15,6 +16,7 @@ import torch
 
 from ..cache.spec import StateSpec
 from ..ops import kernels
+from ..ops.linear import linear
 from ..weights.source import ParamSpec
 from .base import Addend, LayerCache, Mixer, TensorGetter
 from .registry import lookup, register_mixer
@@ -50,6 +52,7 @@ class SideBySide(Mixer):
         if (self.out_norm_eps is not None) != (len(self.out_norms) == 2 and self.hidden_size > 0):
             raise ValueError("norms on the members' results need an eps, two weights' names and the row's size")
         self.norm_weights: Optional[List[torch.Tensor]] = None
+        self.w_in: Optional[torch.Tensor] = None
 
     def cache_spec(self):
         for m in self.members:
@@ -86,6 +89,12 @@ class SideBySide(Mixer):
     def load(self, get: TensorGetter) -> None:
         for m in self.members:
             m.load(get)
+        if all(hasattr(m, "forward_from") and getattr(m, "w_in", None) is not None for m in self.members):
+            self.w_in = torch.cat([m.w_in for m in self.members], dim=0).contiguous()
+            at = 0
+            for m in self.members:                       # the members' matrices are parts of it now
+                m.w_in = self.w_in[at:at + m.w_in.shape[0]]
+                at += m.w_in.shape[0]
         if self.out_norms:
             self.norm_weights = [get(name, "vector").float().contiguous() for name in self.out_norms]
 
@@ -97,11 +106,17 @@ class SideBySide(Mixer):
 
     def _results(self, x, ctx, cache: LayerCache) -> List[torch.Tensor]:
         results = []
+        proj = linear(x, self.w_in, out_dtype=torch.float32) if self.w_in is not None else None
+        at = 0
         for m, span in zip(self.members, self._state_at):
             state = cache.state[:, span[0]:span[1]] if span is not None and cache.state is not None else None
             view = LayerCache(pages=cache.pages if m.cache_spec() is not None else None, group=cache.group, state=state,
                               writes=cache.writes)
-            out, bias = m.forward(x, ctx, view)
+            if proj is not None:
+                out, bias = m.forward_from(proj[:, at:at + m.w_in.shape[0]], ctx, view)
+                at += m.w_in.shape[0]
+            else:
+                out, bias = m.forward(x, ctx, view)
             out = out.float() if out.dtype != torch.float32 else out
             if bias is not None:
                 out = out + bias.float()
